@@ -392,6 +392,8 @@ typedef struct {
     float out_scale;               /* factor on the head outputs (0 is read as 1) */
     const float* elem_gate; int64_t ld_elem_gate;   /* fp32 logits [T, ld_elem_gate] or NULL: output column c of a row (head h at
                                       column h * vdim) is multiplied by sigmoid(elem_gate[row][c]) */
+    int32_t chunk;                 /* > 0: a query sees only keys of its own run of `chunk` positions (position / chunk equal,
+                                      counted from the sequence's start); 0: no runs. May be combined with a window */
 } p3_attn_window_args;
 /* query rows per tile that p3_attn_window_prefill takes for these sizes: 64 on its tensor-core path, else 32 */
 int p3_attn_window_tile_rows(const p3_attn_window_args* args);
@@ -456,6 +458,8 @@ int p3_latent_post(const p3_latent_post_args* args, cudaStream_t st);
 
 /* out (act) [R, F] = silu(g[r][c]) * u[r][c]; g and u fp32 with the common row pitch ld */
 int p3_glu_silu(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, cudaStream_t st);
+/* the same with another activation in front of the product: act 0 = silu, 1 = relu (max(g, 0) * u) */
+int p3_glu_act(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, int act, cudaStream_t st);
 
 /* router with sigmoid scores: z = Wr x (fp32; or logits fp32 [T, ld_logits] when an earlier product already formed them with fp32
  * accumulation: x and Wr are then unused), s = sigmoid(z), choice = s + correction (correction fp32 [E] or NULL). The E
@@ -492,7 +496,8 @@ int p3_token_shift(const float* h, const float* shift, float* state, const int32
 /* After a fused q|k|v projection (proj fp32 [T, ld_proj]; bias fp32 indexed like proj's columns, or NULL): the leading rot_n
  * numbers of every query and key head turn by position * freq[i] (number i paired with i + rot_n / 2, freq fp32 [rot_n / 2]), the
  * rest passes; q -> q_out (act), k -> K pool, v -> V pool. v_off < 0: there is no value projection, the value of a token is its key
- * BEFORE the rotation (vdim == dim). */
+ * BEFORE the rotation (vdim == dim). rot_mag: factor on cos and sin (0 is read as 1). unit_norm != 0: every query and key head is then
+ * divided by its root mean square, sqrt(mean over dim of the squares + eps), after the rotation. */
 typedef struct {
     const float* proj; int64_t ld_proj; int32_t q_off, k_off, v_off;
     const float* bias;
@@ -501,6 +506,7 @@ typedef struct {
     void* k_pool; void* v_pool; const int32_t* block_table; int32_t bt_stride;
     const int32_t* tok_slot; const int32_t* tok_pos; int32_t T;
     int32_t act_f32, cache_f32;
+    float rot_mag; int32_t unit_norm; float eps;
 } p3_qkv_rope_post_args;
 int p3_qkv_rope_post(const p3_qkv_rope_post_args* args, cudaStream_t st);
 
@@ -589,6 +595,57 @@ int p3_gla_scan(const p3_gla_args* args, cudaStream_t st);
 int p3_headnorm_gate_x(const float* y, int64_t ldy, const float* den, int n_heads, int vdim, const float* gain, int gain_shared,
                        const float* gate, int64_t ld_gate, int gate_silu, float scale, float eps, void* out, int64_t ldo, int out_f32,
                        int64_t T, cudaStream_t st);
+
+
+/* ---- parts of decoders with one norm in front of every sublayer, a normed embedding that re-enters at every pass of a looped layer
+ * block, short causal convolutions and a gated delta rule (Lupusun and designs built from these parts) */
+
+/* x fp32 [T, W] = N(table[ids[t]]) * gain with N(v) = v / sqrt(mean(v^2) + eps) (bf16 table); copy (fp32 [T, W] or NULL): the same
+ * rows once more; with gain_pre: h (activation type) = N(x) * gain_pre */
+int p3_embed_norm_rows_f32(const void* table, const int32_t* ids, const float* gain, float* x, float* copy, const float* gain_pre, void* h,
+                           int act_f32, int64_t T, int W, int vocab, float eps, cudaStream_t st);
+
+/* v = x[t] + mult * y[t] (y fp32 [T, ldy] or NULL) + add[t] (fp32 [T, W] or NULL), t = rows ? rows[r] : r. Without `rows` x[t] <- v.
+ * With gain: h[r] (activation type) = v / sqrt(mean(v^2) + eps) * gain. */
+int p3_residual_rmsnorm(float* x, const float* y, int64_t ldy, float mult, const float* add, const int32_t* rows, const float* gain,
+                        void* h, int act_f32, int64_t R, int W, float eps, cudaStream_t st);
+
+/* Short causal convolutions over time, one per channel, silu, and unit length per head; and the gates of a gated delta rule.
+ * Inputs are the columns [c_off, c_off + C) of proj (fp32 [n_rows, ld_proj]), C = n_unit * dim + n_plain:
+ *   z_t[c] = silu(sum_j w[j][c] x_(t - (taps - 1) + j)[c])   (w fp32 [taps][C]; zeros before the start of a sequence)
+ * The leading n_unit heads of dim (<= 512) channels are divided by sqrt(sum of squares + unit_eps), the first n_scaled of them also
+ * multiplied by `scale`. out fp32 [n_rows, ld_out], column c. Inputs of earlier steps come from conv_state fp32
+ * [slots][taps - 1][C] (the last taps - 1 inputs in order of time), which this call only READS: p3_delta_scan advances it.
+ * gates (fp32 [n_rows][n_gates][2] or NULL): {decay, beta} of every head, decay = exp(-exp(a_log) softplus(proj[a_off + h] + dt_bias)),
+ * beta = sigmoid(proj[b_off + h]). */
+typedef struct {
+    const float* proj; int64_t ld_proj; int32_t c_off;
+    int32_t n_unit, dim, n_scaled, n_plain;
+    const float* w; int32_t taps; const float* conv_state;
+    float scale, unit_eps;
+    const int32_t* seqs; const int32_t* slot_seq; const int32_t* tok_slot; int32_t n_rows;
+    float* out; int64_t ld_out;
+    int32_t a_off, b_off, n_gates; const float* a_log; const float* dt_bias; float* gates;
+} p3_short_conv_args;
+int p3_short_conv(const p3_short_conv_args* args, cudaStream_t st);
+
+/* Gated delta rule (csrc/recurrent.cu). Per head a state S [dim][vdim] (dim <= 512), zero at the start of a sequence:
+ *   S <- decay S,  u = beta (v - S^T k),  S <- S + k u^T,  y = S^T q
+ * token by token over the rows of every sequence of `seqs`, fp32. q, k (n_kv x dim) and v (n_heads x vdim) are columns of qkv (fp32
+ * [T, ld_qkv]); head h uses query/key head h / (n_heads / n_kv); gates fp32 [T][n_heads][2] = {decay, beta}. out fp32 [T, ld_out],
+ * head h at column h * vdim. The state of a slot is `state + slot * p3_delta_state_floats(...)` floats, read at the start and written at
+ * the end of the step. With taps > 1 the call also advances the convolution history conv_state (fp32 [slots][taps - 1][channels]) of
+ * every sequence by the step's rows of conv_in (fp32 [T, ld_conv_in], `channels` columns). rs_force as for the matrix memory. */
+typedef struct {
+    const float* qkv; int64_t ld_qkv; int32_t q_off, k_off, v_off;
+    const float* gates;
+    int32_t n_heads, n_kv, dim, vdim;
+    float* state; const int32_t* seqs; int32_t n_seqs;
+    float* out; int64_t ld_out; int32_t rs_force;
+    const float* conv_in; int64_t ld_conv_in; int32_t channels, taps; float* conv_state;
+} p3_delta_scan_args;
+int64_t p3_delta_state_floats(int n_heads, int dim, int vdim);
+int p3_delta_scan(const p3_delta_scan_args* args, cudaStream_t st);
 
 #ifdef __cplusplus
 }

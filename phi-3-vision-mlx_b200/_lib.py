@@ -89,10 +89,15 @@ _SIGS = {
     'p3_embed_pair_rows_f32': [_p, _p, _p, _p, _p, _p, _p, _l, _p, _l, _i, _i, _f, _l, _l, _l, _p],
     'p3_distance_linear_table': [_p, _p, _i, _i, _p],
     'p3_headnorm_gate_x': [_p, _l, _p, _i, _i, _p, _i, _p, _l, _i, _f, _f, _p, _l, _i, _l, _p],
+    # normed embedding, residual add with one norm behind it, gated unit with a choice of activation (csrc/seq_ops.cu)
+    'p3_embed_norm_rows_f32': [_p, _p, _p, _p, _p, _p, _p, _i, _l, _i, _i, _f, _p],
+    'p3_residual_rmsnorm': [_p, _p, _l, _f, _p, _p, _p, _p, _i, _l, _i, _f, _p],
+    'p3_glu_act': [_p, _p, _l, _p, _l, _i, _l, _i, _i, _p],
 }
+GLU_SILU, GLU_RELU = 0, 1                                                 # activations of p3_glu_act
 ROUTER_SOFTMAX, ROUTER_GROUP_MAX, ROUTER_PLAIN_WEIGHTS = 1, 2, 4          # mode bits of p3_router_groups
 _STRUCT_ENTRIES = ['p3_gemm_any', 'p3_qkv_post', 'p3_attn_window_prefill', 'p3_attn_window_decode', 'p3_latent_post',
-                   'p3_qkv_rope_post', 'p3_matrix_memory_scan', 'p3_gla_scan']
+                   'p3_qkv_rope_post', 'p3_matrix_memory_scan', 'p3_gla_scan', 'p3_short_conv', 'p3_delta_scan']
 ATTN_WINDOW_MMA = os.environ.get('P3_ATTN_WINDOW_MMA', '1') != '0'
 
 _lib = None
@@ -102,7 +107,8 @@ launches = 0          # number of p3_* kernel-launching calls issued (bench.py r
 def exported_symbols():
     return sorted(list(_SIGS) + ['p3_last_error', 'p3_version', 'p3_attention_decode_workspace', 'p3_decode_mega',
                                  'p3_decode_mega_ctas', 'p3_gemm_fused', 'p3_gemm_plan_weights', 'p3_gemm_skinny_x', 'p3_trace_set', 'p3_trace_count',
-                                 'p3_attn_window_tile_rows', 'p3_matrix_memory_state_floats', 'p3_gla_state_floats']
+                                 'p3_attn_window_tile_rows', 'p3_matrix_memory_state_floats', 'p3_gla_state_floats',
+                                 'p3_delta_state_floats']
                   + _STRUCT_ENTRIES)
 
 
@@ -126,6 +132,7 @@ def lib():
             L.p3_attn_window_tile_rows.argtypes, L.p3_attn_window_tile_rows.restype = [_p], C.c_int
             L.p3_matrix_memory_state_floats.argtypes, L.p3_matrix_memory_state_floats.restype = [_i, _i, _i], C.c_int64
             L.p3_gla_state_floats.argtypes, L.p3_gla_state_floats.restype = [_i, _i, _i], C.c_int64
+            L.p3_delta_state_floats.argtypes, L.p3_delta_state_floats.restype = [_i, _i, _i], C.c_int64
             L.p3_last_error.restype = C.c_char_p
             L.p3_version.restype = C.c_int
             _lib = L
@@ -146,6 +153,7 @@ def lib():
         L.p3_attn_window_tile_rows.argtypes, L.p3_attn_window_tile_rows.restype = [_p], C.c_int
         L.p3_matrix_memory_state_floats.argtypes, L.p3_matrix_memory_state_floats.restype = [_i, _i, _i], C.c_int64
         L.p3_gla_state_floats.argtypes, L.p3_gla_state_floats.restype = [_i, _i, _i], C.c_int64
+        L.p3_delta_state_floats.argtypes, L.p3_delta_state_floats.restype = [_i, _i, _i], C.c_int64
         _lib = L
     return _lib
 
@@ -241,7 +249,7 @@ class AttnWindowArgs(C.Structure):
                 ('n_heads', C.c_int32), ('n_kv', C.c_int32), ('dim', C.c_int32), ('vdim', C.c_int32), ('scale', C.c_float),
                 ('window', C.c_int32), ('act_f32', C.c_int32), ('cache_f32', C.c_int32), ('tiles', _p), ('n_tiles', C.c_int32),
                 ('n_splits', C.c_int32), ('ws', _p), ('v_ld', C.c_int32), ('keep_first', C.c_int32), ('sig_bias', _p),
-                ('out_scale', C.c_float), ('elem_gate', _p), ('ld_elem_gate', _l)]
+                ('out_scale', C.c_float), ('elem_gate', _p), ('ld_elem_gate', _l), ('chunk', C.c_int32)]
 
 
 class LatentPostArgs(C.Structure):
@@ -263,7 +271,8 @@ class QkvRopePostArgs(C.Structure):
                 ('n_heads', C.c_int32), ('n_kv', C.c_int32), ('dim', C.c_int32), ('vdim', C.c_int32), ('rot_n', C.c_int32),
                 ('freq', _p), ('q_out', _p), ('ld_q', _l),
                 ('k_pool', _p), ('v_pool', _p), ('block_table', _p), ('bt_stride', C.c_int32),
-                ('tok_slot', _p), ('tok_pos', _p), ('T', C.c_int32), ('act_f32', C.c_int32), ('cache_f32', C.c_int32)]
+                ('tok_slot', _p), ('tok_pos', _p), ('T', C.c_int32), ('act_f32', C.c_int32), ('cache_f32', C.c_int32),
+                ('rot_mag', C.c_float), ('unit_norm', C.c_int32), ('eps', C.c_float)]
 
 
 class MatrixMemoryArgs(C.Structure):
@@ -281,3 +290,20 @@ class GlaArgs(C.Structure):
                 ('n_heads', C.c_int32), ('dim', C.c_int32), ('vdim', C.c_int32), ('q_scale', C.c_float),
                 ('state', _p), ('seqs', _p), ('n_seqs', C.c_int32), ('out', _p), ('ld_out', _l), ('rs_force', C.c_int32),
                 ('n_rows', C.c_int32), ('lr', _p), ('ld_lr', _l), ('a2', _p), ('rank', C.c_int32)]
+
+
+class ShortConvArgs(C.Structure):
+    """p3_short_conv_args (include/phi3_b200.h)"""
+    _fields_ = [('proj', _p), ('ld_proj', _l), ('c_off', C.c_int32),
+                ('n_unit', C.c_int32), ('dim', C.c_int32), ('n_scaled', C.c_int32), ('n_plain', C.c_int32),
+                ('w', _p), ('taps', C.c_int32), ('conv_state', _p), ('scale', C.c_float), ('unit_eps', C.c_float),
+                ('seqs', _p), ('slot_seq', _p), ('tok_slot', _p), ('n_rows', C.c_int32), ('out', _p), ('ld_out', _l),
+                ('a_off', C.c_int32), ('b_off', C.c_int32), ('n_gates', C.c_int32), ('a_log', _p), ('dt_bias', _p), ('gates', _p)]
+
+
+class DeltaScanArgs(C.Structure):
+    """p3_delta_scan_args (include/phi3_b200.h)"""
+    _fields_ = [('qkv', _p), ('ld_qkv', _l), ('q_off', C.c_int32), ('k_off', C.c_int32), ('v_off', C.c_int32), ('gates', _p),
+                ('n_heads', C.c_int32), ('n_kv', C.c_int32), ('dim', C.c_int32), ('vdim', C.c_int32),
+                ('state', _p), ('seqs', _p), ('n_seqs', C.c_int32), ('out', _p), ('ld_out', _l), ('rs_force', C.c_int32),
+                ('conv_in', _p), ('ld_conv_in', _l), ('channels', C.c_int32), ('taps', C.c_int32), ('conv_state', _p)]

@@ -140,6 +140,32 @@ def tiny_tagenex(width=96, vocab=300, layers=None, eps=1e-5):
     return {'architecture': 'Tagenex', 'vocab': vocab, 'width': width, 'norm': {'eps': eps}, 'layers': layers}
 
 
+# ------------------------------------------------------------------------------------------------ parsing that designs share
+def layer_runs(loop, n):
+    """config entry {"start", "stop", "times"} (or None) and the number of layers -> (the entry as a namespace or None, the layer runs
+    in order: (layer index, does a pass of the looped block start with this run)). Layers start .. stop - 1 run `times` times in a
+    row."""
+    if not loop:
+        return None, [(i, False) for i in range(n)]
+    lo, hi, times = int(loop['start']), int(loop['stop']), int(loop['times'])
+    if not (0 <= lo < hi <= n and times >= 1):
+        raise ValueError('loop: need 0 <= start < stop <= layers and times >= 1')
+    order = list(range(lo)) + list(range(lo, hi)) * times + list(range(hi, n))
+    return SimpleNamespace(start=lo, stop=hi, times=times), [(i, i == lo) for i in order]
+
+
+def scaled_rotation(i, r, width, what):
+    """config entry {"base", "dims", "scaling": {"factor", "original", "fast", "slow"} or absent} of layer i -> namespace for
+    yarn_frequencies; `width`: how many numbers of a head may turn (the default of dims), `what`: its name in the config"""
+    sc = r.get('scaling')
+    rot = SimpleNamespace(base=float(r['base']), dims=int(r.get('dims', width)),
+                          scaling=None if not sc else SimpleNamespace(factor=float(sc['factor']), original=float(sc['original']),
+                                                                      fast=float(sc['fast']), slow=float(sc['slow'])))
+    if rot.dims % 2 or not 0 < rot.dims <= width:
+        raise ValueError(f'layer {i}: rot.dims must be even and at most {what}')
+    return rot
+
+
 # ------------------------------------------------------------------------------------------------ Tapalix
 class TapalixConfig:
     """config.json of a Tapalix checkpoint: {"architecture": "Tapalix", "vocab", "width", "norm": {"eps"}, "embedding": {"scale"},
@@ -170,14 +196,7 @@ class TapalixConfig:
                                     vdim=int(m.get('vdim', m['dim'])), kv_rank=int(m['kv_rank']), scale=float(m['scale']),
                                     rot_dim=int(m.get('rot_dim', 0)) if rotary else 0, rot=None)
             if rotary and mixer.rot_dim > 0:
-                r = m['rot']
-                sc = r.get('scaling')
-                mixer.rot = SimpleNamespace(base=float(r['base']), dims=int(r.get('dims', mixer.rot_dim)),
-                                            scaling=None if not sc else SimpleNamespace(
-                                                factor=float(sc['factor']), original=float(sc['original']),
-                                                fast=float(sc['fast']), slow=float(sc['slow'])))
-                if mixer.rot.dims % 2 or not 0 < mixer.rot.dims <= mixer.rot_dim:
-                    raise ValueError(f'layer {i}: rot.dims must be even and at most rot_dim')
+                mixer.rot = scaled_rotation(i, m['rot'], mixer.rot_dim, 'rot_dim')
             f = lc.get('mlp')
             if f is None:
                 ff = None
@@ -196,18 +215,9 @@ class TapalixConfig:
             else:
                 raise NotImplementedError(f"layer {i}: feed-forward kind {f['kind']!r}")
             self.layers.append(SimpleNamespace(mixer=mixer, ff=ff))
-        self.num_hidden_layers = n = len(self.layers)
-        lp = d.get('loop')
-        if lp:
-            lo, hi, times = int(lp['start']), int(lp['stop']), int(lp['times'])
-            if not (0 <= lo < hi <= n and times >= 1):
-                raise ValueError('loop: need 0 <= start < stop <= layers and times >= 1')
-            self.loop = SimpleNamespace(start=lo, stop=hi, times=times)
-            order = list(range(lo)) + list(range(lo, hi)) * times + list(range(hi, n))
-        else:
-            self.loop, lo, order = None, -1, list(range(n))
+        self.num_hidden_layers = len(self.layers)
         # (layer index, does a pass of the loop start with this run)
-        self.runs = [(i, i == lo) for i in order]
+        self.loop, self.runs = layer_runs(d.get('loop'), len(self.layers))
 
     def kv_layout(self):
         """per layer RUN (one shared head, latent + turning key numbers, no separate values): what the page pool allocates"""
@@ -497,4 +507,86 @@ def tiny_danalorn(width=96, vocab=300, layers=None, eps=1e-5, bigram=(257, 29, 5
          'layers': layers}
     if bigram:
         d['embedding']['bigram'] = {'buckets': bigram[0], 'mul_prev': bigram[1], 'mul_cur': bigram[2]}
+    return d
+
+
+# ------------------------------------------------------------------------------------------------ Lupusun
+class LupusunConfig:
+    """config.json of a Lupusun checkpoint: {"architecture": "Lupusun", "vocab", "width", "norm": {"eps"}, "residual_mult", "layers":
+    [...], "loop": {"start", "stop", "times"} or absent}. A layer entry has "type", "mixer" and "mlp":
+      type "delta":     mixer = {heads, kv_heads, dim, vdim, conv}: gated delta rule behind short convolutions of `conv` taps, query and
+                        key heads (of dim numbers) shared by groups of value heads (of vdim);
+      type "attention": mixer = {heads, kv_heads, dim, vdim, scale, mask: {size}, rot: {base, dims, scaling: {factor, original, fast,
+                        slow}}}: biased projections, a partial rotation with blended frequencies, unit heads after it, keys of the
+                        query's own chunk of `size` positions, a learned per-head sink;
+      mlp: null | {"kind": "dense", ff}: a gated relu unit.
+    Absent optional keys mean: no chunks, no rotation, plain frequencies, no loop. Nothing is assumed equal between layers. `runs` lists
+    the layer runs in order (a looped layer once per pass): every run has a cache or a state of its own."""
+    UNIT_EPS = 1e-6              # under the root of the unit length of the recurrence's queries and keys: fixed by the design
+
+    def __init__(self, d):
+        self.raw = d
+        self.architecture = d.get('architecture', 'Lupusun')
+        self.architectures = [self.architecture]
+        self.vocab_size, self.width = int(d['vocab']), int(d['width'])
+        self.eps = float(d['norm']['eps'])
+        self.residual_mult = float(d.get('residual_mult', 1.0))
+        self.layers = []
+        for i, lc in enumerate(d['layers']):
+            kind, m = lc.get('type'), lc['mixer']
+            if kind not in ('delta', 'attention'):
+                raise NotImplementedError(f'layer {i}: mixer type {kind!r} is not part of this design')
+            mixer = SimpleNamespace(kind=kind, heads=int(m['heads']), kv_heads=int(m.get('kv_heads', m['heads'])), dim=int(m['dim']),
+                                    vdim=int(m.get('vdim', m['dim'])))
+            if mixer.heads % mixer.kv_heads:
+                raise ValueError(f'layer {i}: heads must be a multiple of kv_heads')
+            if kind == 'delta':
+                mixer.taps = int(m['conv'])
+                if mixer.taps < 1:
+                    raise ValueError(f'layer {i}: the convolutions need at least one tap')
+                if not 1 <= mixer.dim <= 512:
+                    raise NotImplementedError(f'layer {i}: key size {mixer.dim} of the recurrence; the kernels take 1 .. 512')
+            else:
+                mixer.scale, mixer.chunk = float(m['scale']), int((m.get('mask') or {}).get('size') or 0)
+                r = m.get('rot')
+                mixer.rot = scaled_rotation(i, r, mixer.dim, 'dim') if r and int(r.get('dims', mixer.dim)) != 0 else None
+                if mixer.chunk < 0:
+                    raise ValueError(f'layer {i}: mask.size must not be negative')
+                if mixer.dim > 4096 or mixer.vdim > 4096:
+                    raise NotImplementedError(f'layer {i}: head sizes above 4096; the attention kernels take at most that')
+            f = lc.get('mlp')
+            if f is None:
+                ff = None
+            elif f['kind'] == 'dense':
+                ff = SimpleNamespace(kind='dense', ff=int(f['ff']))
+            else:
+                raise NotImplementedError(f"layer {i}: feed-forward kind {f['kind']!r}")
+            self.layers.append(SimpleNamespace(mixer=mixer, ff=ff))
+        self.num_hidden_layers = len(self.layers)
+        self.loop, self.runs = layer_runs(d.get('loop'), len(self.layers))
+
+    def kv_layout(self):
+        """per layer RUN (kv heads, key size, value size): what the page pool allocates; a recurrent layer caches nothing"""
+        mixers = [self.layers[i].mixer for i, _ in self.runs]
+        return [(m.kv_heads, m.dim, m.vdim) if m.kind == 'attention' else (0, 0, 0) for m in mixers]
+
+
+def tiny_lupusun(width=96, vocab=300, layers=None, loop=(1, 3, 2), eps=1e-5, residual_mult=0.8):
+    """A small Lupusun config dict for tests: sizes deliberately unequal between layers (dim != vdim, heads != kv_heads, partly rotated
+    heads, chunks that differ and one layer without, convolutions of four and of three taps), one layer without a feed-forward; layers 1
+    and 2 run twice."""
+    att = lambda heads, kv, dim, vdim, chunk, rd, factor=4.0, base=10000.0: {
+        'type': 'attention',
+        'mixer': dict(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, scale=2.0 * dim ** -0.5, **({'mask': {'size': chunk}} if chunk else {}),
+                      rot={'base': base, 'dims': rd, **({'scaling': {'factor': factor, 'original': 64, 'fast': 16.0, 'slow': 1.5}} if factor else {})})}
+    delta = lambda heads, kv, dim, vdim, taps: {'type': 'delta', 'mixer': dict(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, conv=taps)}
+    dense = lambda ff: {'kind': 'dense', 'ff': ff}
+    if layers is None:
+        layers = [dict(delta(4, 2, 24, 40, 4), mlp=dense(136)),
+                  dict(att(6, 3, 40, 24, 50, 16), mlp=dense(72)),
+                  dict(delta(3, 3, 40, 16, 3), mlp=None),
+                  dict(att(4, 1, 24, 56, 0, 24, factor=None), mlp=dense(88))]
+    d = {'architecture': 'Lupusun', 'vocab': vocab, 'width': width, 'norm': {'eps': eps}, 'residual_mult': residual_mult, 'layers': layers}
+    if loop:
+        d['loop'] = {'start': loop[0], 'stop': loop[1], 'times': loop[2]}
     return d

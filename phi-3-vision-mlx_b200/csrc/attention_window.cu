@@ -1,6 +1,7 @@
 // Paged attention over a ragged batch with a sliding window, a per-head sink in the softmax denominator and a per-head distance
 // penalty: score(i, j) = scale * q_i . k_j - pen[h][i - j], visible when 0 <= i - j < window (window 0: every earlier key),
-// weights = exp(score) / (exp(sink_h) + sum over visible exp(score)); optional output gates per (token, head) and per output number
+// weights = exp(score) / (exp(sink_h) + sum over visible exp(score)); with `chunk` a query sees only keys of its own run of `chunk`
+// positions, counted from the start of the sequence; optional output gates per (token, head) and per output number
 // (the sigmoid of a logit, applied in the epilogue). Head sizes of
 // keys (dim) and values (vdim) are independent run-time numbers, grouped-query heads share K/V (head h reads h / (H/G)). The fp32
 // kernels take any size (rows above 256 numbers in key chunks and value column blocks), the tensor-core kernels sizes up to 256.
@@ -37,12 +38,21 @@ __device__ __forceinline__ float elem_gate(const p3_attn_window_args& a, size_t 
 constexpr int BQ = 32, WARPS = 4, RPW = BQ / WARPS;          // prefill: query rows per CTA / per warp
 constexpr int WIDE = 256;                                    // fp32 kernels: key numbers per chunk, value columns per CTA
 
+// first position that a query at `pos` sees (kept first tokens aside): the start of its window, the start of its chunk, or 0. It
+// never falls as pos grows.
+__device__ __forceinline__ int first_key(const p3_attn_window_args& a, int pos) {
+    int lo = 0;
+    if (a.window > 0) lo = max(lo, pos - a.window + 1);
+    if (a.chunk > 0) lo = max(lo, pos - pos % a.chunk);
+    return lo;
+}
+
 // The pages a tile of queries visits: those of the kept first tokens that lie before the window's pages, then the pages from
-// the first key inside the first row's window to the last row's own position.
+// the first key the first row sees to the last row's own position.
 struct PageWalk {
     int keep, n_keep, lo, n;
     __device__ PageWalk(const p3_attn_window_args& a, int first, int last) {
-        keep = a.window > 0 ? a.keep_first : 0;              // without a window every earlier key is visible anyway
+        keep = a.keep_first;                                 // without a limit every earlier key is visible anyway (first = 0)
         lo = first / P3_PAGE;
         n_keep = min((keep + P3_PAGE - 1) / P3_PAGE, lo);
         n = n_keep + last / P3_PAGE - lo + 1;
@@ -78,14 +88,16 @@ __global__ void __launch_bounds__(WARPS * 32) attn_window_prefill_kernel(p3_attn
     if (nchunk == 1) stage_q(0, d);
     const float sink = a.sink ? a.sink[h] : -FLT_MAX;
     float m[RPW], l[RPW], acc[RPW][DVC];
+    int lo[RPW];                                             // first visible key of the row
 #pragma unroll
     for (int r = 0; r < RPW; r++) {
+        lo[r] = first_key(a, pos0 + warp * RPW + r);
         m[r] = sink; l[r] = a.sink ? 1.f : 0.f;
 #pragma unroll
         for (int j = 0; j < DVC; j++) acc[r][j] = 0.f;
     }
     const int last = pos0 + nq - 1;
-    const int first = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+    const int first = first_key(a, pos0);
     const int32_t* bt = a.block_table + (size_t)slot * a.bt_stride;
     const float* pen = a.penalty ? a.penalty + (size_t)h * a.n_penalty : nullptr;
     const bool sig = a.sig_bias != nullptr;                  // sigmoid weights: no running maximum, no denominator
@@ -133,7 +145,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_window_prefill_kernel(p3_attn
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int kpos = pg * P3_PAGE + lane + 32 * e, dist = qpos - kpos;
-                const bool vis = qr < nq && dist >= 0 && (a.window <= 0 || dist < a.window || kpos < walk.keep);
+                const bool vis = qr < nq && dist >= 0 && (kpos >= lo[r] || kpos < walk.keep);
                 float v = -FLT_MAX;
                 if (vis) v = s[r][e] - (pen ? pen[min(dist, a.n_penalty - 1)] : 0.f);
                 pv[e] = v;
@@ -224,7 +236,7 @@ __device__ __forceinline__ void stage_rows(bf16* dst, int ld, const bf16* src, i
 // registers, in the base-2 domain (scale, penalty and sink carry the factor log2 e, so a weight is one subtraction and one
 // ex2); the weights are rounded to bf16 only as the A operand of P.V, taken straight from the score accumulators. K fragments
 // come by ldmatrix from the row-major page, V by ldmatrix.trans. A page that every row of the tile sees in full (behind the
-// diagonal, inside the window) skips the visibility tests.
+// diagonal, inside the window and the chunk) skips the visibility tests.
 template <int DK, int DN, int MINB, bool SIG>
 __global__ void __launch_bounds__(128, MINB) attn_window_prefill_mma_kernel(p3_attn_window_args a) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
@@ -245,11 +257,12 @@ __global__ void __launch_bounds__(128, MINB) attn_window_prefill_mma_kernel(p3_a
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
     const int r0 = warp * 16 + gid, r1 = r0 + 8;             // this thread's two rows of the tile
     const int last = pos0 + nq - 1;
-    const int first = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+    const int first = first_key(a, pos0);
     const int32_t* bt = a.block_table + (size_t)slot * a.bt_stride;
     const float* pen = a.penalty ? a.penalty + (size_t)h * a.n_penalty : nullptr;
     const int kc = d / 8, vc = dv / 8;                       // 16-byte chunks per row
     const PageWalk walk(a, first, last);
+    const int lo0 = first_key(a, pos0 + r0), lo1 = first_key(a, pos0 + r1), lo_last = first_key(a, last);   // first visible keys
     constexpr bool sig = SIG;                                // sigmoid weights (a.sig_bias): no running maximum, no denominator
     const float sbias2 = sig ? a.sig_bias[h] * LOG2E : 0.f;
 
@@ -316,8 +329,8 @@ __global__ void __launch_bounds__(128, MINB) attn_window_prefill_mma_kernel(p3_a
             }
         }
         float mx0 = -FLT_MAX, mx1 = -FLT_MAX;
-        // every key of the page is visible to every row of the tile: behind the first row, and the last row's window reaches it
-        const bool full = pg * P3_PAGE + 63 <= pos0 && (a.window <= 0 || pos0 + 63 - pg * P3_PAGE < a.window || pg * P3_PAGE + 63 < walk.keep);
+        // every key of the page is visible to every row of the tile: behind the first row, and the last row still sees it
+        const bool full = pg * P3_PAGE + 63 <= pos0 && (pg * P3_PAGE >= lo_last || pg * P3_PAGE + 63 < walk.keep);
         // the penalty depends on row - col only, and this thread's second row is its first plus 8: the penalties of (r1, key block
         // j) are those of (r0, key block j - 1), so 18 values serve the 32 scores
         float pq[9][2];
@@ -340,7 +353,7 @@ __global__ void __launch_bounds__(128, MINB) attn_window_prefill_mma_kernel(p3_a
                 for (int e = 0; e < 4; e++) {
                     const int row = (e < 2) ? r0 : r1, col = j * 8 + tig * 2 + (e & 1);
                     const int kpos = pg * P3_PAGE + col, dist = pos0 + row - kpos;
-                    const bool vis = row < nq && dist >= 0 && (a.window <= 0 || dist < a.window || kpos < walk.keep);
+                    const bool vis = row < nq && dist >= 0 && (kpos >= ((e < 2) ? lo0 : lo1) || kpos < walk.keep);
                     s[j][e] = vis ? fmaf(s[j][e], scale2, -pq[(e < 2) ? j + 1 : j][e & 1]) : -FLT_MAX;
                 }
         }
@@ -460,9 +473,9 @@ __global__ void __launch_bounds__(DW * 32) attn_window_decode_kernel(p3_attn_win
     const int row = tile.x, slot = tile.z, pos = tile.w;
     const int g = blockIdx.y / v_parts, split = blockIdx.z, n_splits = gridDim.z;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int first = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int first = first_key(a, pos);
     // the visible keys in one running index: the kept first tokens that lie before the window, then the window
-    const int n_keep = a.window > 0 ? min(a.keep_first, first) : 0, n_vis = n_keep + pos - first + 1;
+    const int n_keep = min(a.keep_first, first), n_vis = n_keep + pos - first + 1;
     const int per = ((n_vis + n_splits - 1) / n_splits + 31) & ~31;
     const int k_lo = split * per, k_hi = min(n_vis, k_lo + per);
     auto key_at = [&](int c) { return c < n_keep ? c : first + c - n_keep; };
@@ -639,7 +652,7 @@ __global__ void __launch_bounds__(128, 2) attn_window_decode_mma_kernel(p3_attn_
     const int row = tile.x, slot = tile.z, pos = tile.w;
     const int g = PARTS ? blockIdx.y / v_parts : blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
-    const int first = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int first = first_key(a, pos);
     const PageWalk walk(a, first, pos);                      // the kept first pages, then the window's pages: one running index
     const int per = (walk.n + n_splits - 1) / n_splits;      // pages per slice, rounded up
     const int pg_lo = split * per;                           // first running index of this slice
@@ -847,7 +860,7 @@ int check_args(const p3_attn_window_args* a, const char* who) {
     P3_CHECK_ARG(!a->penalty || a->n_penalty >= 1, "%s: empty penalty table", who);
     P3_CHECK_ARG(a->act_f32 == a->cache_f32, "%s: activations and cache must both be fp32 or both bf16", who);
     P3_CHECK_ARG(a->v_ld == 0 || a->v_ld >= a->vdim, "%s: the value row pitch must hold a value row", who);
-    P3_CHECK_ARG(a->keep_first >= 0, "%s: keep_first must not be negative", who);
+    P3_CHECK_ARG(a->keep_first >= 0 && a->chunk >= 0, "%s: keep_first and chunk must not be negative", who);
     P3_CHECK_ARG(!a->sig_bias || !a->sink, "%s: sigmoid weights have no denominator for a sink", who);
     return 0;
 }

@@ -35,6 +35,17 @@
 //                               round ahead) with a staged row of decays beside every k and q row. There is no normaliser and no
 //                               stabiliser (every factor is in (0, 1]), so all four warps own columns. As there, a token's
 //                               arithmetic does not depend on how the sequence was cut into steps.
+//
+// Gated delta rule (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule"). Per head a state S [dim][vdim]
+// that starts at zero, one decay g and one step size b per head and token:
+//     S <- g_t S        u_t = b_t (v_t - S^T k_t)        S <- S + k_t u_t^T        y_t = S^T q_t
+//   short_conv_kernel           what precedes the recurrence, over all rows of the step at once: a causal convolution of a few taps per
+//                               channel, silu, unit length per query / key head, and the gates g and b of every head. A warp owns the
+//                               channels of one head (or a block of value channels) and walks a few rows with its last inputs in
+//                               registers; inputs of earlier steps come from the slot's history, which it only reads
+//   delta_scan_kernel           the layout of the linear-attention scan; two passes over the state columns per token, the sums S^T k
+//                               (a shuffle reduction closes them, on the critical path) and then update and read-out. It also moves the
+//                               convolution history on: by then no kernel of the step reads the old one.
 #include "common.cuh"
 #include "../../include/phi3_b200.h"
 #include <cfloat>
@@ -415,6 +426,269 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) gla_scan_kernel(p3_gla_args a)
             if (col + c * CW < dv && d0 + j < d) Sg[(size_t)(d0 + j) * dv + col + c * CW] = S[c][j];
 }
 
+// ---------------------------------------------------------------- short convolutions, unit heads, gates of the delta rule
+template <int VEC> __device__ __forceinline__ void ldvec(const float* p, float* v) {
+    if constexpr (VEC == 4) { const float4 u = *reinterpret_cast<const float4*>(p); v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w; }
+    else if constexpr (VEC == 2) { const float2 u = *reinterpret_cast<const float2*>(p); v[0] = u.x; v[1] = u.y; }
+    else v[0] = *p;
+}
+template <int VEC> __device__ __forceinline__ void stvec(float* p, const float* v) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else if constexpr (VEC == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+    else *p = v[0];
+}
+
+// A lane owns NV vectors of VEC neighbouring channels, 32 VEC apart. TAPS > 0: the last TAPS - 1 inputs stay in registers from row
+// to row; TAPS 0: any number of taps, every row reads its inputs again.
+template <int VEC, int NV, int TAPS>
+__global__ void __launch_bounds__(128) short_conv_kernel(p3_short_conv_args a, int rows_per, int n_conv_jobs) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    constexpr int N = VEC * NV, WB = 32 * N, WIN = TAPS > 1 ? TAPS - 1 : 1;
+    const int lane = threadIdx.x & 31, job = blockIdx.y * 4 + (threadIdx.x >> 5);
+    const int taps = TAPS > 0 ? TAPS : a.taps;
+    const int C = a.n_unit * a.dim + a.n_plain;
+    const int r_lo = blockIdx.x * rows_per, r_hi = min(a.n_rows, r_lo + rows_per);
+    if (job >= n_conv_jobs) {                                // gates: {decay, beta} of every head
+        if (job > n_conv_jobs || !a.gates) return;
+        for (int i = lane; i < (r_hi - r_lo) * a.n_gates; i += 32) {
+            const int r = r_lo + i / a.n_gates, h = i % a.n_gates;
+            const float* pr = a.proj + (size_t)r * a.ld_proj;
+            const float z = pr[a.a_off + h] + a.dt_bias[h], b = pr[a.b_off + h];
+            const float soft = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));              // softplus without overflow
+            float* g = a.gates + ((size_t)r * a.n_gates + h) * 2;
+            g[0] = expf(-expf(a.a_log[h]) * soft);
+            g[1] = 1.0f / (1.0f + expf(-b));
+        }
+        return;
+    }
+    const bool unit = job < a.n_unit;
+    const int c0 = unit ? job * a.dim : a.n_unit * a.dim + (job - a.n_unit) * WB;
+    const int width = unit ? a.dim : min(WB, C - c0);
+    const float scale = unit && job < a.n_scaled ? a.scale : 1.f;
+    const float* in = a.proj + a.c_off + c0;
+    auto load = [&](const float* p, float* v) {              // the lane's channels of one row (zeros beyond the width)
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (k * 32 + lane) * VEC;
+            if (i < width) ldvec<VEC>(p + i, v + k * VEC);
+            else
+#pragma unroll
+                for (int e = 0; e < VEC; e++) v[k * VEC + e] = 0.f;
+        }
+    };
+    float w[TAPS > 0 ? TAPS : 1][N], win[WIN][N], cur[N], nxt[N];
+    if (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) load(a.w + (size_t)j * C + c0, w[j]);
+    }
+    int seq_lo = 0, seq_hi = 0, slot = 0, pos0 = 0;          // the sequence the row belongs to: its rows of this step, slot, first position
+    // the input `back` rows before row r of the batch: from the step's rows, from the slot's history, or zero before the start
+    auto load_back = [&](int r, int back, float* v) {
+        const int rel = r - seq_lo - back;                   // row of the sequence in this step; negative: an earlier step
+        if (rel >= 0) load(in + (size_t)(r - back) * a.ld_proj, v);
+        else if (pos0 + rel >= 0) load(a.conv_state + ((size_t)slot * (taps - 1) + (taps - 1 + rel)) * C + c0, v);
+        else
+#pragma unroll
+            for (int e = 0; e < N; e++) v[e] = 0.f;
+    };
+    if (r_lo < r_hi) load(in + (size_t)r_lo * a.ld_proj, cur);
+    for (int r = r_lo; r < r_hi; r++) {
+        if (r + 1 < r_hi) load(in + (size_t)(r + 1) * a.ld_proj, nxt);
+        if (r >= seq_hi) {                                   // another sequence begins (or this warp's first row)
+            const int4 rec = reinterpret_cast<const int4*>(a.seqs)[a.slot_seq[a.tok_slot[r]]];   // {first row, rows, slot, first position}
+            seq_lo = rec.x; seq_hi = rec.x + rec.y; slot = rec.z; pos0 = rec.w;
+            if (TAPS > 1) {
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; j++) load_back(r, TAPS - 1 - j, win[j]);
+            }
+        }
+        float z[N];
+#pragma unroll
+        for (int e = 0; e < N; e++) z[e] = 0.f;
+        if (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; j++)
+#pragma unroll
+                for (int e = 0; e < N; e++) z[e] = fmaf(w[j][e], win[j][e], z[e]);
+#pragma unroll
+            for (int e = 0; e < N; e++) z[e] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][e], cur[e], z[e]);
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; j++)
+#pragma unroll
+                for (int e = 0; e < N; e++) win[j][e] = j + 2 < TAPS ? win[j + 1 < WIN ? j + 1 : 0][e] : cur[e];
+        } else {
+            for (int j = 0; j < taps; j++) {
+                float x[N], wj[N];
+                load_back(r, taps - 1 - j, x);
+                load(a.w + (size_t)j * C + c0, wj);
+#pragma unroll
+                for (int e = 0; e < N; e++) z[e] = fmaf(wj[e], x[e], z[e]);
+            }
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < N; e++) { z[e] = z[e] / (1.0f + expf(-z[e])); ss = fmaf(z[e], z[e], ss); }   // silu; channels beyond the width stay 0
+        if (unit) {
+            const float f = scale / sqrtf(warp_sum(ss) + a.unit_eps);
+#pragma unroll
+            for (int e = 0; e < N; e++) z[e] *= f;
+        }
+        float* o = a.out + (size_t)r * a.ld_out + c0;
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (k * 32 + lane) * VEC;
+            if (i < width) stvec<VEC>(o + i, z + k * VEC);
+        }
+#pragma unroll
+        for (int e = 0; e < N; e++) cur[e] = nxt[e];
+    }
+}
+
+// ---------------------------------------------------------------- gated delta rule
+// a 16-byte shared load that the compiler does not merge with an earlier one of the same address
+__device__ __forceinline__ float4 lds_again(const float4* p) {
+    float4 v;
+    asm volatile("ld.shared.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(smem_u32(p)));
+    return v;
+}
+
+__host__ __device__ inline int64_t delta_head_floats(int dim, int vdim) { return (int64_t)dim * vdim; }
+
+template <int DS, int RS, int NC, int TB>
+__global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_scan_args a) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    // a warp = RS row slices x CW lanes, every lane with NC columns (CW apart); DP: dim rounded up
+    constexpr int CW = 32 / RS, WCOLS = CW * NC, COLS = GLA_WARPS * WCOLS, DP = DS * RS;
+    constexpr int NT = GLA_WARPS * 32;
+    constexpr int DPP = DP + 4 * RS;                         // pitch of a staged row: its RS slices 4 floats apart (bank spread)
+    constexpr int ROUND = TB * (2 * DPP + COLS + 2);         // floats of one staged round
+    auto at_row = [](int c) { return c + 4 * (c / DS); };    // where number c of a row lives
+    extern __shared__ __align__(16) float sm[];
+    const int d = a.dim, dv = a.vdim, H = a.n_heads;
+    // two rounds in flight: [q [TB][DPP] (zeros beyond dim) | k alike | v [TB][COLS] | {decay, beta} [TB]]
+    const int4 rec = reinterpret_cast<const int4*>(a.seqs)[blockIdx.x];
+    const int row0 = rec.x, n_tok = rec.y, slot = rec.z, pos0 = rec.w;
+    const int hd = blockIdx.y, hk = hd / (H / a.n_kv), vb = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const bool fresh = pos0 == 0;
+    float* Sg = a.state + ((size_t)slot * H + hd) * delta_head_floats(d, dv);
+    const int col = vb * COLS + warp * WCOLS + lane % CW, d0 = (lane / CW) * DS;   // first of this lane's columns
+    const bool vec = d % 4 == 0 && a.ld_qkv % 4 == 0 && a.q_off % 4 == 0 && a.k_off % 4 == 0 && ((uintptr_t)a.qkv & 15) == 0;
+
+    // all threads: start the copies of the round that begins at token t0 into buffer `buf`
+    auto stage = [&](int t0, int buf) {
+        const int nb = min(TB, n_tok - t0);
+        float* qs = sm + buf * ROUND;
+        float* ks = qs + TB * DPP;
+        float* vs = ks + TB * DPP;
+        float* gs = vs + TB * COLS;
+        if (vec) {
+            for (int i = tid; i < nb * (DP / 4); i += NT) {
+                const int tt = i / (DP / 4), c = (i - tt * (DP / 4)) * 4;
+                const float* pr = a.qkv + (size_t)(row0 + t0 + tt) * a.ld_qkv + (size_t)hk * d + (c < d ? c : 0);
+                cp_async16(smem_u32(qs + tt * DPP + at_row(c)), pr + a.q_off, c < d ? 16 : 0);
+                cp_async16(smem_u32(ks + tt * DPP + at_row(c)), pr + a.k_off, c < d ? 16 : 0);
+            }
+        } else {
+            for (int i = tid; i < nb * DP; i += NT) {
+                const int tt = i / DP, c = i - tt * DP;
+                const float* pr = a.qkv + (size_t)(row0 + t0 + tt) * a.ld_qkv + (size_t)hk * d + (c < d ? c : 0);
+                cp_async4z(smem_u32(qs + tt * DPP + at_row(c)), pr + a.q_off, c < d ? 4 : 0);
+                cp_async4z(smem_u32(ks + tt * DPP + at_row(c)), pr + a.k_off, c < d ? 4 : 0);
+            }
+        }
+        for (int i = tid; i < nb * COLS; i += NT) {
+            const int tt = i / COLS, c = vb * COLS + (i - tt * COLS);
+            cp_async4z(smem_u32(vs + i), a.qkv + (size_t)(row0 + t0 + tt) * a.ld_qkv + a.v_off + (size_t)hd * dv + (c < dv ? c : 0), c < dv ? 4 : 0);
+        }
+        for (int i = tid; i < nb * 2; i += NT) cp_async4z(smem_u32(gs + i), a.gates + ((size_t)(row0 + t0 + i / 2) * H + hd) * 2 + (i & 1), 4);
+    };
+
+    stage(0, 0);
+    cp_async_commit();
+    // the convolution history moves on by this sequence's rows: channel by channel in order of time, so that a history longer than
+    // the step's rows can shift in place
+    if (a.taps > 1) {
+        const int keep = a.taps - 1, n_thr = NT * gridDim.y * gridDim.z;
+        float* hist = a.conv_state + (size_t)slot * keep * a.channels;
+        for (int c = (blockIdx.z * gridDim.y + blockIdx.y) * NT + tid; c < a.channels; c += n_thr)
+            for (int j = 0; j < keep; j++) {
+                const int rel = n_tok - keep + j;            // row of the step; negative: an entry of the old history
+                hist[(size_t)j * a.channels + c] = rel >= 0 ? a.conv_in[(size_t)(row0 + rel) * a.ld_conv_in + c]
+                                                            : pos0 + rel >= 0 ? hist[(size_t)(j + n_tok) * a.channels + c] : 0.f;
+            }
+    }
+    float S[NC][DS];
+#pragma unroll
+    for (int c = 0; c < NC; c++)
+#pragma unroll
+        for (int j = 0; j < DS; j++)
+            S[c][j] = (!fresh && col + c * CW < dv && d0 + j < d) ? Sg[(size_t)(d0 + j) * dv + col + c * CW] : 0.f;
+    for (int t0 = 0, r = 0; t0 < n_tok; t0 += TB, r++) {
+        const int nb = min(TB, n_tok - t0), buf = r & 1;
+        cp_async_wait<0>();                                  // this thread's copies of round r have landed ...
+        __syncthreads();                                     // ... and everyone's; round r - 1 is consumed
+        if (t0 + TB < n_tok) stage(t0 + TB, buf ^ 1);
+        cp_async_commit();
+        const float* qs = sm + buf * ROUND;
+        const float* ks = qs + TB * DPP;
+        const float* vs = ks + TB * DPP;
+        const float* gs = vs + TB * COLS;
+#pragma unroll(DS >= 64 ? 1 : 2)
+        for (int tt = 0; tt < nb; tt++) {
+            const float keep = gs[2 * tt], beta = gs[2 * tt + 1];
+            const float4* kq = reinterpret_cast<const float4*>(ks + tt * DPP + at_row(d0));
+            const float4* qq = reinterpret_cast<const float4*>(qs + tt * DPP + at_row(d0));
+            float acc[NC][4], u[NC];
+#pragma unroll
+            for (int c = 0; c < NC; c++) acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
+#pragma unroll
+            for (int j = 0; j < DS; j += 4) {
+                const float4 kk = kq[j / 4];
+#pragma unroll
+                for (int c = 0; c < NC; c++) {
+                    acc[c][0] = fmaf(S[c][j], kk.x, acc[c][0]);         acc[c][1] = fmaf(S[c][j + 1], kk.y, acc[c][1]);
+                    acc[c][2] = fmaf(S[c][j + 2], kk.z, acc[c][2]);     acc[c][3] = fmaf(S[c][j + 3], kk.w, acc[c][3]);
+                }
+            }
+#pragma unroll
+            for (int c = 0; c < NC; c++) {
+                float p = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
+                if (RS >= 2) p += __shfl_xor_sync(0xffffffffu, p, CW);
+                if (RS >= 4) p += __shfl_xor_sync(0xffffffffu, p, 2 * CW);
+                u[c] = beta * (vs[tt * COLS + warp * WCOLS + lane % CW + c * CW] - keep * p);   // (decay S)^T k = decay (S^T k)
+                acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
+            }
+#pragma unroll
+            for (int j = 0; j < DS; j += 4) {
+                // up to 32 rows per lane the k row stays in registers between the passes
+                const float4 kk = DS <= 32 ? kq[j / 4] : lds_again(kq + j / 4), qv = qq[j / 4];
+#pragma unroll
+                for (int c = 0; c < NC; c++) {
+                    S[c][j] = fmaf(kk.x, u[c], keep * S[c][j]);         acc[c][0] = fmaf(S[c][j], qv.x, acc[c][0]);
+                    S[c][j + 1] = fmaf(kk.y, u[c], keep * S[c][j + 1]); acc[c][1] = fmaf(S[c][j + 1], qv.y, acc[c][1]);
+                    S[c][j + 2] = fmaf(kk.z, u[c], keep * S[c][j + 2]); acc[c][2] = fmaf(S[c][j + 2], qv.z, acc[c][2]);
+                    S[c][j + 3] = fmaf(kk.w, u[c], keep * S[c][j + 3]); acc[c][3] = fmaf(S[c][j + 3], qv.w, acc[c][3]);
+                }
+            }
+#pragma unroll
+            for (int c = 0; c < NC; c++) {
+                float y = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
+                if (RS >= 2) y += __shfl_xor_sync(0xffffffffu, y, CW);
+                if (RS >= 4) y += __shfl_xor_sync(0xffffffffu, y, 2 * CW);
+                if (lane < CW && col + c * CW < dv)
+                    a.out[(size_t)(row0 + t0 + tt) * a.ld_out + (size_t)hd * dv + col + c * CW] = y;
+            }
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < NC; c++)
+#pragma unroll
+        for (int j = 0; j < DS; j++)
+            if (col + c * CW < dv && d0 + j < d) Sg[(size_t)(d0 + j) * dv + col + c * CW] = S[c][j];
+}
+
 // one warp per (token, head)
 template <typename AT>
 __global__ void headnorm_gate_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ den, int H, int dv,
@@ -564,5 +838,65 @@ extern "C" int p3_gla_scan(const p3_gla_args* a, cudaStream_t st) {
     else { if (ds == 16) GO(16, 4, 2); else if (ds == 32) GO(32, 4, 2); else GO(64, 4, 2); }
 #undef GO
     P3_CHECK_LAUNCH("gla_scan");
+    return 0;
+}
+
+extern "C" int p3_short_conv(const p3_short_conv_args* a, cudaStream_t st) {
+    P3_CHECK_ARG(a && a->proj && a->w && a->seqs && a->slot_seq && a->tok_slot && a->out, "short_conv: null argument");
+    P3_CHECK_ARG(a->taps >= 1 && (a->taps == 1 || a->conv_state), "short_conv: several taps need the history");
+    P3_CHECK_ARG(a->n_unit >= 0 && a->n_plain >= 0 && a->n_scaled <= a->n_unit && (a->n_unit == 0 || (a->dim >= 1 && a->dim <= 512)),
+                 "short_conv: need 1 <= dim <= 512 and n_scaled <= n_unit");
+    P3_CHECK_ARG(!a->gates || (a->n_gates >= 1 && a->a_log && a->dt_bias), "short_conv: the gates need a_log and dt_bias");
+    P3_CHECK_ARG(((uintptr_t)a->seqs & 15) == 0, "short_conv: the sequence records must be 16-byte aligned");
+    if (a->n_rows == 0) return 0;
+    const int d = a->n_unit ? a->dim : 128, C = a->n_unit * a->dim + a->n_plain;
+    auto fits = [&](int v) {                                 // may a lane take v neighbouring channels at once?
+        const uintptr_t m = (uintptr_t)v * 4 - 1;
+        return d % v == 0 && C % v == 0 && a->c_off % v == 0 && a->ld_proj % v == 0 && a->ld_out % v == 0 &&
+               (((uintptr_t)a->proj | (uintptr_t)a->w | (uintptr_t)a->out | (uintptr_t)a->conv_state) & m) == 0;
+    };
+    const int vec = d > 64 && fits(4) ? 4 : d > 32 && fits(2) ? 2 : 1;
+    const int need = (d + 32 * vec - 1) / (32 * vec), nv = need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : need <= 8 ? 8 : 16;
+    const int wb = 32 * vec * nv, conv_jobs = a->n_unit + (a->n_plain + wb - 1) / wb, jobs = conv_jobs + (a->gates ? 1 : 0);
+    const int rows_per = a->n_rows >= 512 ? 16 : a->n_rows >= 128 ? 4 : 1;
+    const dim3 grid((unsigned)((a->n_rows + rows_per - 1) / rows_per), (unsigned)((jobs + 3) / 4));
+#define GO(V, N)                                                                                                               \
+    do { if (a->taps == 4) p3_launch_pdl(short_conv_kernel<V, N, 4>, dim3(grid), dim3(128), (size_t)(0), st, *a, rows_per, conv_jobs); \
+         else p3_launch_pdl(short_conv_kernel<V, N, 0>, dim3(grid), dim3(128), (size_t)(0), st, *a, rows_per, conv_jobs); } while (0)
+    if (vec == 4) { if (nv == 1) GO(4, 1); else if (nv == 2) GO(4, 2); else GO(4, 4); }
+    else if (vec == 2) { if (nv == 1) GO(2, 1); else if (nv == 2) GO(2, 2); else if (nv == 4) GO(2, 4); else GO(2, 8); }
+    else { if (nv == 1) GO(1, 1); else if (nv == 2) GO(1, 2); else if (nv == 4) GO(1, 4); else if (nv == 8) GO(1, 8); else GO(1, 16); }
+#undef GO
+    P3_CHECK_LAUNCH("short_conv");
+    return 0;
+}
+
+extern "C" int64_t p3_delta_state_floats(int n_heads, int dim, int vdim) { return (int64_t)n_heads * delta_head_floats(dim, vdim); }
+
+extern "C" int p3_delta_scan(const p3_delta_scan_args* a, cudaStream_t st) {
+    P3_CHECK_ARG(a && a->qkv && a->gates && a->state && a->seqs && a->out, "delta_scan: null argument");
+    P3_CHECK_ARG(a->n_heads >= 1 && a->n_kv >= 1 && a->n_heads % a->n_kv == 0, "delta_scan: heads must be a multiple of kv heads");
+    P3_CHECK_ARG(a->dim >= 1 && a->dim <= 512 && a->vdim >= 1, "delta_scan: need 1 <= dim <= 512, vdim >= 1");
+    P3_CHECK_ARG(a->taps <= 1 || (a->conv_in && a->conv_state && a->channels >= 1), "delta_scan: the convolution history needs its inputs");
+    P3_CHECK_ARG(((uintptr_t)a->seqs & 15) == 0, "delta_scan: the sequence records must be 16-byte aligned");
+    if (a->n_seqs == 0) return 0;
+    // A warp is four row slices x eight lanes, a lane owns one or two columns: the choice of the linear-attention scan
+    int rs = 4, nc = (int64_t)a->n_seqs * a->n_heads * ((a->vdim + 31) / 32) > 148 ? 2 : 1;
+    if (a->rs_force == 2 || a->rs_force == 4) { rs = a->rs_force; nc = 1; }
+    if (a->rs_force == 8) { rs = 4; nc = 2; }
+    if (a->dim > 256) { rs = 4; nc = 1; }                    // 128 rows per thread, 16 tokens per round
+    const int per = (a->dim + rs - 1) / rs, ds = per <= 16 ? 16 : per <= 32 ? 32 : per <= 64 ? 64 : 128;
+    const int cols = GLA_WARPS * 32 / rs * nc, tb = a->dim > 256 ? 16 : MM_TB;
+    const dim3 grid((unsigned)a->n_seqs, (unsigned)a->n_heads, (unsigned)((a->vdim + cols - 1) / cols));
+    const size_t bytes = sizeof(float) * (size_t)2 * tb * (2 * (ds * rs + 4 * rs) + cols + 2);   // two staged rounds
+#define GO(DS, RS, NC, TB)                                                                                             \
+    do { if (set_smem_attr(delta_scan_kernel<DS, RS, NC, TB>, bytes)) return -1;                                         \
+         p3_launch_pdl(delta_scan_kernel<DS, RS, NC, TB>, dim3(grid), dim3(GLA_WARPS * 32), (size_t)(bytes), st, *a); } while (0)
+    if (a->dim > 256) GO(128, 4, 1, 16);
+    else if (rs == 2) { if (ds == 16) GO(16, 2, 1, MM_TB); else if (ds == 32) GO(32, 2, 1, MM_TB); else if (ds == 64) GO(64, 2, 1, MM_TB); else GO(128, 2, 1, MM_TB); }
+    else if (nc == 1) { if (ds == 16) GO(16, 4, 1, MM_TB); else if (ds == 32) GO(32, 4, 1, MM_TB); else GO(64, 4, 1, MM_TB); }
+    else { if (ds == 16) GO(16, 4, 2, MM_TB); else if (ds == 32) GO(32, 4, 2, MM_TB); else GO(64, 4, 2, MM_TB); }
+#undef GO
+    P3_CHECK_LAUNCH("delta_scan");
     return 0;
 }

@@ -510,24 +510,25 @@ __global__ void latent_post_kernel(p3_latent_post_args a) {
     }
 }
 
-// ---------------------------------------------------------------- y = silu(g) * u
-template <typename AT>
-__global__ void glu_silu_kernel(const float* __restrict__ g, const float* __restrict__ u, int64_t ld, AT* __restrict__ out, int64_t ldo,
-                                int64_t R, int F) {
+// ---------------------------------------------------------------- y = act(g) * u, act = silu or relu
+template <int ACT> __device__ __forceinline__ float glu_act(float g) { return ACT == 0 ? g / (1.0f + expf(-g)) : fmaxf(g, 0.f); }
+
+template <typename AT, int ACT>
+__global__ void glu_kernel(const float* __restrict__ g, const float* __restrict__ u, int64_t ld, AT* __restrict__ out, int64_t ldo,
+                           int64_t R, int F) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
     pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
     const int64_t n = R * F;
     for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
         const int64_t r = i / F; const int c = (int)(i % F);
-        const float gv = g[(size_t)r * ld + c], uv = u[(size_t)r * ld + c];
-        stv(out + (size_t)r * ldo + c, gv / (1.0f + expf(-gv)) * uv);
+        stv(out + (size_t)r * ldo + c, glu_act<ACT>(g[(size_t)r * ld + c]) * u[(size_t)r * ld + c]);
     }
 }
 
 // four columns per thread (F, the row pitches and the pointers are multiples of four elements): 16-byte loads
-template <typename AT>
-__global__ void glu_silu_vec4_kernel(const float* __restrict__ g, const float* __restrict__ u, int64_t ld, AT* __restrict__ out,
-                                     int64_t ldo, int64_t R, int F) {
+template <typename AT, int ACT>
+__global__ void glu_vec4_kernel(const float* __restrict__ g, const float* __restrict__ u, int64_t ld, AT* __restrict__ out,
+                                int64_t ldo, int64_t R, int F) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
     pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
     const int F4 = F / 4;
@@ -535,8 +536,8 @@ __global__ void glu_silu_vec4_kernel(const float* __restrict__ g, const float* _
     for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
         const int64_t r = i / F4; const int c = (int)(i % F4) * 4;
         const float4 gv = *reinterpret_cast<const float4*>(g + (size_t)r * ld + c), uv = *reinterpret_cast<const float4*>(u + (size_t)r * ld + c);
-        const float y0 = gv.x / (1.0f + expf(-gv.x)) * uv.x, y1 = gv.y / (1.0f + expf(-gv.y)) * uv.y;
-        const float y2 = gv.z / (1.0f + expf(-gv.z)) * uv.z, y3 = gv.w / (1.0f + expf(-gv.w)) * uv.w;
+        const float y0 = glu_act<ACT>(gv.x) * uv.x, y1 = glu_act<ACT>(gv.y) * uv.y;
+        const float y2 = glu_act<ACT>(gv.z) * uv.z, y3 = glu_act<ACT>(gv.w) * uv.w;
         AT* o = out + (size_t)r * ldo + c;
         if constexpr (sizeof(AT) == 4) *reinterpret_cast<float4*>(o) = make_float4(y0, y1, y2, y3);
         else *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(y0, y1), pack_bf16(y2, y3));
@@ -737,20 +738,29 @@ __global__ void token_shift_kernel(const float* __restrict__ h, const float* __r
     }
 }
 
-// ---------------------------------------------------------------- rotation of q and k + paged K/V write (+ projection biases)
+// ---------------------------------------------------------------- rotation of q and k + paged K/V write (+ projection biases, unit norm)
 // Grid (token, job group): one warp per head job (H query heads, G key heads, G value heads when there is a value projection).
-// The lane that owns number i < rot_n / 2 of a head also owns its partner i + rot_n / 2; angles are position * frequency in fp32
-// with the full-range sincosf. Without a value projection the key head is written twice: rotated to the K pool, as projected to
-// the V pool.
+// The CTA forms cos and sin of its token's angles once, in shared memory: position * frequency in fp32 with the full-range
+// sincosf. The lane that owns number i < rot_n / 2 of a head also owns its partner i + rot_n / 2. Without a value projection the
+// key head is written twice: rotated to the K pool, as projected to the V pool. The root mean square of the unit norm is taken
+// from the numbers before they turn: a rotation keeps the length of a pair, so its squares count with the factor mag^2.
 template <typename AT, typename CT>
 __global__ void qkv_rope_kv_write_kernel(p3_qkv_rope_post_args a) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
     pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    extern __shared__ float2 turn[];                         // [rot_n / 2] {cos, sin} * mag
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const float* pr = a.proj + (size_t)t * a.ld_proj;
     const int slot = a.tok_slot[t], pos = a.tok_pos[t];
     const int page = a.block_table[(size_t)slot * a.bt_stride + pos / P3_PAGE], off = pos % P3_PAGE;
     const int H = a.n_heads, G = a.n_kv, d = a.dim, dv = a.vdim, half = a.rot_n / 2;
+    const float mag = a.rot_mag != 0.f ? a.rot_mag : 1.f;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)pos * a.freq[i], &sn, &cs);
+        turn[i] = make_float2(cs * mag, sn * mag);
+    }
+    __syncthreads();
     const bool v_is_k = a.v_off < 0;
     const int jobs = H + G + (v_is_k ? 0 : G);
     for (int job = blockIdx.y * nw + warp; job < jobs; job += gridDim.y * nw) {
@@ -763,19 +773,27 @@ __global__ void qkv_rope_kv_write_kernel(p3_qkv_rope_post_args a) {
             AT* dq = isq ? (AT*)a.q_out + (size_t)t * a.ld_q + (size_t)h * d : nullptr;
             CT* dk = isq ? nullptr : (CT*)a.k_pool + (((size_t)page * G + h) * P3_PAGE + off) * d;
             CT* dvv = (!isq && v_is_k) ? (CT*)a.v_pool + (((size_t)page * G + h) * P3_PAGE + off) * dv : nullptr;
+            float r = 1.f;
+            if (a.unit_norm) {
+                float st = 0.f, sp = 0.f;                    // squares of the turning and of the passing numbers
+                for (int i = lane; i < d; i += 32) {
+                    const float u = src[i] + (b ? b[i] : 0.f);
+                    if (i < a.rot_n) st = fmaf(u, u, st); else sp = fmaf(u, u, sp);
+                }
+                r = 1.0f / sqrtf(warp_sum(fmaf(st, mag * mag, sp)) / (float)d + a.eps);
+            }
             for (int i = lane; i < d; i += 32) {
                 if (i >= half && i < a.rot_n) continue;      // the partner of a turning pair: written by the pair's owner
                 const float u = src[i] + (b ? b[i] : 0.f);
                 if (i < half) {
                     const float w = src[i + half] + (b ? b[i + half] : 0.f);
-                    float sn, cs;
-                    sincosf((float)pos * a.freq[i], &sn, &cs);
-                    const float r0 = u * cs - w * sn, r1 = w * cs + u * sn;
+                    const float cs = turn[i].x, sn = turn[i].y;
+                    const float r0 = (u * cs - w * sn) * r, r1 = (w * cs + u * sn) * r;
                     if (isq) { stv(dq + i, r0); stv(dq + i + half, r1); }
                     else { stv(dk + i, r0); stv(dk + i + half, r1); if (dvv) { stv(dvv + i, u); stv(dvv + i + half, w); } }
                 } else {
-                    if (isq) stv(dq + i, u);
-                    else { stv(dk + i, u); if (dvv) stv(dvv + i, u); }
+                    if (isq) stv(dq + i, u * r);
+                    else { stv(dk + i, u * r); if (dvv) stv(dvv + i, u); }
                 }
             }
         } else {
@@ -924,6 +942,130 @@ __global__ void embed_pair_rows_kernel(const bf16* __restrict__ table, const bf1
         }
 #pragma unroll
         for (int k = 0; k < RPT; k++) { const int i = i0 + k * blockDim.x; if (i < W) x[(size_t)t * W + i] = v[k] * scale + u[k]; }
+    }
+}
+
+// ---------------------------------------------------------------- rows of RPT * blockDim numbers in registers, VEC at a time
+// number k of a thread's register row (k < RPT) is element row_at<VEC>(k); VEC neighbours are loaded and stored together
+template <int VEC> __device__ __forceinline__ int row_at(int k) { return ((k / VEC) * blockDim.x + threadIdx.x) * VEC + k % VEC; }
+
+template <int VEC> __device__ __forceinline__ void row_load(const float* p, int W, float* v) {
+#pragma unroll
+    for (int k = 0; k < RPT; k += VEC) {
+        const int i = row_at<VEC>(k);
+        if constexpr (VEC == 4) {
+            const float4 u = i < W ? *reinterpret_cast<const float4*>(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[k] = u.x; v[k + 1] = u.y; v[k + 2] = u.z; v[k + 3] = u.w;
+        } else v[k] = i < W ? p[i] : 0.f;
+    }
+}
+template <int VEC, typename AT> __device__ __forceinline__ void row_store(AT* p, int W, const float* v) {
+#pragma unroll
+    for (int k = 0; k < RPT; k += VEC) {
+        const int i = row_at<VEC>(k);
+        if (i >= W) continue;
+        if constexpr (VEC == 4 && sizeof(AT) == 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[k], v[k + 1], v[k + 2], v[k + 3]);
+        else if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p + i) = make_uint2(pack_bf16(v[k], v[k + 1]), pack_bf16(v[k + 2], v[k + 3]));
+        else stv(p + i, v[k]);
+    }
+}
+
+// ---------------------------------------------------------------- embedding row under a norm (+ copy, + the first layer's norm of it)
+template <typename AT, int VEC>
+__global__ void embed_norm_rows_kernel(const bf16* __restrict__ table, const int32_t* __restrict__ ids, const float* __restrict__ gain,
+                                       float* __restrict__ x, float* __restrict__ copy, const float* __restrict__ gpre, AT* __restrict__ h,
+                                       int W, int vocab, float eps) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    __shared__ float sh[32];
+    const int64_t t = blockIdx.x;
+    int id = ids[t];
+    if (id < 0 || id >= vocab) id = 0;
+    const bf16* src = table + (size_t)id * W;
+    const int nt = blockDim.x;
+    float v[RPT], gv[RPT];
+#pragma unroll
+    for (int k = 0; k < RPT; k += VEC) {
+        const int i = row_at<VEC>(k);
+        if constexpr (VEC == 4) {
+            const uint2 u = i < W ? *reinterpret_cast<const uint2*>(src + i) : make_uint2(0u, 0u);
+            const float2 lo = unpack_bf16(u.x), hi = unpack_bf16(u.y);
+            v[k] = lo.x; v[k + 1] = lo.y; v[k + 2] = hi.x; v[k + 3] = hi.y;
+        } else v[k] = i < W ? __bfloat162float(src[i]) : 0.f;
+    }
+    row_load<VEC>(gain, W, gv);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < RPT; k++) ss = fmaf(v[k], v[k], ss);
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) { const float u = __bfloat162float(src[i]); ss = fmaf(u, u, ss); }
+    ss = block_sum(ss, sh);
+    const float r = 1.0f / sqrtf(ss / (float)W + eps);
+    float s2 = 0.f;
+#pragma unroll
+    for (int k = 0; k < RPT; k++) { v[k] = v[k] * r * gv[k]; s2 = fmaf(v[k], v[k], s2); }
+    row_store<VEC>(x + (size_t)t * W, W, v);
+    if (copy) row_store<VEC>(copy + (size_t)t * W, W, v);
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) {
+        const float u = __bfloat162float(src[i]) * r * gain[i];
+        x[(size_t)t * W + i] = u;
+        if (copy) copy[(size_t)t * W + i] = u;
+        s2 = fmaf(u, u, s2);
+    }
+    if (!gpre) return;
+    row_load<VEC>(gpre, W, gv);
+    s2 = block_sum(s2, sh);
+    const float r2 = 1.0f / sqrtf(s2 / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < RPT; k++) v[k] = v[k] * r2 * gv[k];
+    row_store<VEC>(h + (size_t)t * W, W, v);
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) stv(h + (size_t)t * W + i, x[(size_t)t * W + i] * r2 * gpre[i]);   // this thread's own write
+}
+
+// ---------------------------------------------------------------- x += mult * y (+ add) ; h = rms_norm(x) * gain
+template <typename AT, int VEC>
+__global__ void residual_rmsnorm_kernel(float* x, const float* __restrict__ y, int64_t ldy, float mult, const float* __restrict__ add,
+                                        const int32_t* __restrict__ rows, const float* __restrict__ gain, AT* __restrict__ h, int W,
+                                        float eps) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    __shared__ float sh[32];
+    const int64_t r = blockIdx.x, t = rows ? rows[r] : r;
+    float* xr = x + (size_t)t * W;
+    const float* yr = y ? y + (size_t)t * ldy : nullptr;
+    const float* ar = add ? add + (size_t)t * W : nullptr;
+    const int nt = blockDim.x;
+    float v[RPT], u[RPT], gv[RPT];
+    row_load<VEC>(xr, W, v);
+    if (yr) {
+        row_load<VEC>(yr, W, u);
+#pragma unroll
+        for (int k = 0; k < RPT; k++) v[k] = fmaf(mult, u[k], v[k]);
+    }
+    if (ar) {
+        row_load<VEC>(ar, W, u);
+#pragma unroll
+        for (int k = 0; k < RPT; k++) v[k] += u[k];
+    }
+    if (gain) row_load<VEC>(gain, W, gv);
+    auto val = [&](int i) { float s = xr[i]; if (yr) s = fmaf(mult, yr[i], s); if (ar) s += ar[i]; return s; };
+    const bool store_x = !rows && (yr || ar);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < RPT; k++) ss = fmaf(v[k], v[k], ss);
+    if (store_x) row_store<VEC>(xr, W, v);
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) { const float s = val(i); ss = fmaf(s, s, ss); }
+    float sc = 0.f;
+    if (gain) {
+        ss = block_sum(ss, sh);
+        sc = 1.0f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+        for (int k = 0; k < RPT; k++) v[k] = v[k] * sc * gv[k];
+        row_store<VEC>(h + (size_t)r * W, W, v);
+    }
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) {   // numbers beyond the registers: formed again, written last
+        const float s = val(i);
+        if (store_x) xr[i] = s;
+        if (gain) stv(h + (size_t)r * W + i, s * sc * gain[i]);
     }
 }
 
@@ -1079,20 +1221,26 @@ extern "C" int p3_latent_post(const p3_latent_post_args* a, cudaStream_t st) {
     return 0;
 }
 
-extern "C" int p3_glu_silu(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F,
-                           cudaStream_t st) {
+extern "C" int p3_glu_act(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, int act,
+                          cudaStream_t st) {
+    P3_CHECK_ARG(act == 0 || act == 1, "glu_act: the activation is 0 (silu) or 1 (relu)");
     if (R == 0 || F == 0) return 0;
     const bool vec = F % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)g & 15) == 0 && ((uintptr_t)u & 15) == 0 &&
                      ((uintptr_t)out & 15) == 0;
     const int64_t n = vec ? R * (F / 4) : R * F;
     const unsigned grid = (unsigned)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-    if (vec) {
-        if (out_f32) p3_launch_pdl(glu_silu_vec4_kernel<float>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (float*)out, ldo, R, F);
-        else p3_launch_pdl(glu_silu_vec4_kernel<bf16>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (bf16*)out, ldo, R, F);
-    } else if (out_f32) p3_launch_pdl(glu_silu_kernel<float>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (float*)out, ldo, R, F);
-    else p3_launch_pdl(glu_silu_kernel<bf16>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (bf16*)out, ldo, R, F);
-    P3_CHECK_LAUNCH("glu_silu");
+#define GO(K, AT) do { if (act == 0) p3_launch_pdl(K<AT, 0>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (AT*)out, ldo, R, F);   \
+                       else p3_launch_pdl(K<AT, 1>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (AT*)out, ldo, R, F); } while (0)
+    if (vec) { if (out_f32) GO(glu_vec4_kernel, float); else GO(glu_vec4_kernel, bf16); }
+    else { if (out_f32) GO(glu_kernel, float); else GO(glu_kernel, bf16); }
+#undef GO
+    P3_CHECK_LAUNCH("glu_act");
     return 0;
+}
+
+extern "C" int p3_glu_silu(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F,
+                           cudaStream_t st) {
+    return p3_glu_act(g, u, ld, out, ldo, out_f32, R, F, 0, st);
 }
 
 extern "C" int p3_router_sigmoid_groups(const void* x, int64_t ldx, int x_f32, const float* Wr, const float* correction,
@@ -1169,12 +1317,14 @@ extern "C" int p3_qkv_rope_post(const p3_qkv_rope_post_args* a, cudaStream_t st)
     P3_CHECK_ARG(a && a->proj && a->q_out && a->k_pool && a->v_pool && a->block_table && a->tok_slot && a->tok_pos, "qkv_rope_post: null argument");
     P3_CHECK_ARG(a->rot_n >= 0 && a->rot_n % 2 == 0 && a->rot_n <= a->dim && (a->rot_n == 0 || a->freq), "qkv_rope_post: rot_n must be even and <= dim, with frequencies");
     P3_CHECK_ARG(a->v_off >= 0 || a->vdim == a->dim, "qkv_rope_post: keys that double as values need vdim == dim");
+    P3_CHECK_ARG(a->rot_n <= 8192, "qkv_rope_post: at most 8192 turning numbers per head");
     if (a->T == 0) return 0;
     const int jobs = a->n_heads + a->n_kv + (a->v_off < 0 ? 0 : a->n_kv), th = 128;
     const int groups = a->T >= 1024 ? 1 : (jobs + 3) / 4;
     const dim3 grid((unsigned)a->T, (unsigned)groups);
-    if (a->act_f32 && a->cache_f32) p3_launch_pdl(qkv_rope_kv_write_kernel<float, float>, dim3(grid), dim3(th), (size_t)(0), st, *a);
-    else if (!a->act_f32 && !a->cache_f32) p3_launch_pdl(qkv_rope_kv_write_kernel<bf16, bf16>, dim3(grid), dim3(th), (size_t)(0), st, *a);
+    const size_t sm = (size_t)(a->rot_n / 2) * sizeof(float2);
+    if (a->act_f32 && a->cache_f32) p3_launch_pdl(qkv_rope_kv_write_kernel<float, float>, dim3(grid), dim3(th), sm, st, *a);
+    else if (!a->act_f32 && !a->cache_f32) p3_launch_pdl(qkv_rope_kv_write_kernel<bf16, bf16>, dim3(grid), dim3(th), sm, st, *a);
     else P3_CHECK_ARG(false, "qkv_rope_post: activations and cache must both be fp32 or both bf16");
     P3_CHECK_LAUNCH("qkv_rope_post");
     return 0;
@@ -1230,5 +1380,35 @@ extern "C" int p3_distance_linear_table(const float* slope, float* pen, int H, i
     const int64_t tot = (int64_t)H * n;
     distance_linear_kernel<<<(unsigned)((tot + 255) / 256), 256, 0, st>>>(slope, pen, H, n);
     P3_CHECK_LAUNCH("distance_linear_table");
+    return 0;
+}
+
+extern "C" int p3_embed_norm_rows_f32(const void* table, const int32_t* ids, const float* gain, float* x, float* copy, const float* gain_pre,
+                                      void* h, int act_f32, int64_t T, int W, int vocab, float eps, cudaStream_t st) {
+    P3_CHECK_ARG(table && ids && gain && x && (!gain_pre || h), "embed_norm_rows_f32: null argument");
+    if (T == 0) return 0;
+    const int th = W > 4096 ? 1024 : W > 2048 ? 512 : W >= 1024 ? 256 : 128;     // the row fits the threads' registers up to W = 8192
+    const bool vec = W % 4 == 0 && (((uintptr_t)gain | (uintptr_t)x | (uintptr_t)copy | (uintptr_t)gain_pre | (uintptr_t)h) & 15) == 0 &&
+                     ((uintptr_t)table & 7) == 0;
+#define GO(AT, V) p3_launch_pdl(embed_norm_rows_kernel<AT, V>, dim3((unsigned)T), dim3(th), (size_t)(0), st, (const bf16*)table, ids, gain, x, copy, gain_pre, (AT*)h, W, vocab, eps)
+    if (act_f32) { if (vec) GO(float, 4); else GO(float, 1); }
+    else { if (vec) GO(bf16, 4); else GO(bf16, 1); }
+#undef GO
+    P3_CHECK_LAUNCH("embed_norm_rows_f32");
+    return 0;
+}
+
+extern "C" int p3_residual_rmsnorm(float* x, const float* y, int64_t ldy, float mult, const float* add, const int32_t* rows,
+                                   const float* gain, void* h, int act_f32, int64_t R, int W, float eps, cudaStream_t st) {
+    P3_CHECK_ARG(x && W >= 1 && (!gain || h), "residual_rmsnorm: null argument");
+    if (R == 0) return 0;
+    const int th = W > 4096 ? 1024 : W > 2048 ? 512 : W >= 1024 ? 256 : 128;
+    const bool vec = W % 4 == 0 && (!y || ldy % 4 == 0) &&
+                     (((uintptr_t)x | (uintptr_t)y | (uintptr_t)add | (uintptr_t)gain | (uintptr_t)h) & 15) == 0;
+#define GO(AT, V) p3_launch_pdl(residual_rmsnorm_kernel<AT, V>, dim3((unsigned)R), dim3(th), (size_t)(0), st, x, y, ldy, mult, add, rows, gain, (AT*)h, W, eps)
+    if (act_f32) { if (vec) GO(float, 4); else GO(float, 1); }
+    else { if (vec) GO(bf16, 4); else GO(bf16, 1); }
+#undef GO
+    P3_CHECK_LAUNCH("residual_rmsnorm");
     return 0;
 }

@@ -35,14 +35,13 @@ Precision. dtype=bfloat16 (serving): matrices, activations that feed a matrix pr
 positions, angles, scores, softmax, norms, the residual sum, decays and their logarithms, the recurrent state and its sums are fp32.
 dtype=float32: everything is fp32 on the FMA pipes (no TF32).
 """
-import ctypes as C
 import os
 
 import torch
 from . import _lib
 from ._lib import call, call_struct, ptr
 from .configs import DanalornConfig
-from .lm_base import PagedLM, _page_slices, _stream
+from .lm_base import PagedLM, _stream
 
 
 class DanalornB200(PagedLM):
@@ -63,11 +62,6 @@ class DanalornB200(PagedLM):
         mat = lambda t: t.to(self.dev, dtype).contiguous()                     # matrices: the compute type
         f32 = lambda t: t.to(self.dev, torch.float32).contiguous()            # everything that enters fp32 arithmetic
         b16 = lambda t: t.to(self.dev, torch.bfloat16).contiguous()
-
-        def rows16(parts):
-            """stacked projection rows, padded with zero rows to a multiple of 16 (small batches keep the weight-streaming kernel)"""
-            n = sum(p.shape[0] for p in parts)
-            return mat(torch.cat(parts + ([torch.zeros(-n % 16, parts[0].shape[1], dtype=parts[0].dtype, device=parts[0].device)] if n % 16 else []), 0))
 
         def expect(name, shape):
             if name not in w:
@@ -102,7 +96,7 @@ class DanalornB200(PagedLM):
                     expect(a + 'dkv', (R + dr, W))
                     parts.append(w[a + 'dkv'])
                     L['c_gain'] = f32(w[a + 'dkv.norm'])
-                L['in_w'] = rows16(parts)
+                L['in_w'] = self.stacked_rows(parts)
                 L['cq_gain'], L['uq'] = f32(w[a + 'dq.norm']), mat(w[a + 'uq'])
                 # the key up-projection is folded into the query: per head [kv_rank, dim]; the value up-projection stays [vdim, kv_rank]
                 L['uk_t'] = mat(w[a + 'uk'].view(H, d, R).transpose(1, 2))
@@ -112,18 +106,18 @@ class DanalornB200(PagedLM):
                     L['freq'], L['rot_n'] = torch.tensor(fr, dtype=torch.float64).to(self.dev, torch.float32), m.rot.dims
                 else:
                     L['freq'], L['rot_n'] = None, 0
-                L['tile_rows'] = self._attention_tile_rows(H, 1, R + dr, R, R + dr)
+                L['tile_rows'] = self.attention_tile_rows(H, 1, R + dr, R, R + dr)
             elif m.kind == 'attention':
                 H, G, d, dv = m.heads, m.kv_heads, m.dim, m.vdim
                 expect(a + 'q', (H * d, W)); expect(a + 'k', (G * d, W)); expect(a + 'v', (G * dv, W)); expect(a + 'g', (H * dv, W))
                 expect(a + 'o', (W, H * dv)); expect(a + 'q.norm', (d,)); expect(a + 'k.norm', (d,))
-                L['in_w'] = rows16([w[a + 'q'], w[a + 'k'], w[a + 'v'], w[a + 'g']])
+                L['in_w'] = self.stacked_rows([w[a + 'q'], w[a + 'k'], w[a + 'v'], w[a + 'g']])
                 L['in_b'] = torch.cat([f32(w[a + 'q.b']), f32(w[a + 'k.b']), f32(w[a + 'v.b'])])
                 L['q_gain'], L['k_gain'], L['out_w'] = f32(w[a + 'q.norm']), f32(w[a + 'k.norm']), mat(w[a + 'o'])
                 L['slope'] = torch.tensor(cfg.slopes(H), dtype=torch.float64).to(self.dev, torch.float32)
                 L['sink'] = torch.zeros(H, dtype=torch.float32, device=self.dev)           # exp(0) = the one in the denominator
                 L['pen'] = None
-                L['tile_rows'] = self._attention_tile_rows(H, G, d, dv, 0)
+                L['tile_rows'] = self.attention_tile_rows(H, G, d, dv, 0)
             else:
                 H, d, dv = m.heads, m.dim, m.vdim
                 expect(a + 'q', (H * d, W)); expect(a + 'k', (H * d, W)); expect(a + 'v', (H * dv, W)); expect(a + 'g', (H * dv, W))
@@ -133,7 +127,7 @@ class DanalornB200(PagedLM):
                 # decay ranks up to 64: the down projection's rows ride in the layer's input product and the scan's first launch forms
                 # the logits from them (fp32); above that the two decay projections are products of their own
                 L['rank'], L['fused_decay'] = r, r <= 64 and os.environ.get('P3_GLA_FUSED_DECAY', '1') != '0'
-                L['in_w'] = rows16([w[a + 'q'], w[a + 'k'], w[a + 'v'], w[a + 'g']] + ([w[a + 'a1']] if L['fused_decay'] else []))
+                L['in_w'] = self.stacked_rows([w[a + 'q'], w[a + 'k'], w[a + 'v'], w[a + 'g']] + ([w[a + 'a1']] if L['fused_decay'] else []))
                 if L['fused_decay']:
                     L['a2_32'] = f32(w[a + 'a2'])
                 else:
@@ -152,15 +146,6 @@ class DanalornB200(PagedLM):
         # kernel (csrc/attention_window.cu), else 32
         self.q_tile = min(L['tile_rows'] for L in self.layers)
         self._pen_len = 0
-
-    def _attention_tile_rows(self, H, G, key, val, v_ld):
-        """query rows per prefill tile that the attention launch takes for these sizes (64: its tensor-core kernels); asked of the
-        library itself so that the engine's tiles and the kernel's choice cannot disagree"""
-        a = _lib.AttnWindowArgs()
-        a.q = a.out = a.k_pool = a.v_pool = a.block_table = a.tiles = 256              # aligned stand-ins: nothing is launched
-        a.ld_q, a.ld_out, a.n_heads, a.n_kv, a.dim, a.vdim, a.v_ld = H * key, H * val, H, G, key, val, v_ld
-        a.act_f32 = a.cache_f32 = self.f32
-        return int(_lib.lib().p3_attn_window_tile_rows(C.byref(a)))
 
     # ------------------------------------------------------------------ what the engine asks of a model
     def kv_layout(self):
@@ -228,35 +213,6 @@ class DanalornB200(PagedLM):
         self.linear(xn, self.head, logits)
         return logits
 
-    def _attend(self, w, L, b, G, key, val, span_of, kv_bytes):
-        """the prefill tiles and the single-token requests of the step through p3_attn_window_*; span_of(n) = keys a query at
-        position n - 1 sees"""
-        st, H = _stream(), w.n_heads
-        esz = 4 if self.f32 else 2
-        if b.n_pf:
-            w.tiles, w.n_tiles = ptr(b.pf_tiles), b.n_pf
-            ev = self._ev()
-            call_struct('p3_attn_window_prefill', w, st)
-            span = span_of(b.max_pos + 1) if w.window else (b.max_pos + 1) // 2
-            self._ev(ev, 'attn_prefill', 2 * (b.T - b.n_dec) * H * span * (key + val), 0)
-        if b.n_dec:
-            w.tiles, w.n_tiles = ptr(b.dec_tiles), b.n_dec
-            span = span_of(b.max_pos + 1)
-            if L['tile_rows'] == 64:
-                if G == 1 and H > 1:
-                    # one shared K/V head: a request is one CTA per slice (two when the values take two column blocks)
-                    w.n_splits = _page_slices(b.n_dec * (-(-val // 128) if key > 128 else 1), 2 * -(-span // 128) + 1, merge=0.4)
-                else:
-                    w.n_splits = _page_slices(b.n_dec * G, 2 * -(-span // 128) + 1)
-            else:
-                # one key per lane: enough CTAs for eight per SM, at least 128 keys (one pass of a CTA) per slice
-                w.n_splits = max(1, min(-(-8 * 148 // (b.n_dec * G)), -(-span // 128)))
-            ws = torch.empty(b.n_dec * H * w.n_splits * (val + 2), dtype=torch.float32, device=self.dev) if w.n_splits > 1 else None
-            w.ws = ptr(ws)
-            ev = self._ev()
-            call_struct('p3_attn_window_decode', w, st)
-            self._ev(ev, 'attn_decode', 2 * b.n_dec * H * span * (key + val), b.n_dec * span * kv_bytes * esz)
-
     def _latent(self, L, li, h, b, pool):
         """normed input h (act [T, W]) -> mixer output before its norm, fp32 [T, W]"""
         st, dev, T, W = _stream(), self.dev, b.T, self.W
@@ -301,7 +257,7 @@ class DanalornB200(PagedLM):
         w.out, w.ld_out, w.sink = ptr(olat), olat.stride(0), ptr(L['sink'])
         w.n_heads, w.n_kv, w.dim, w.vdim, w.scale, w.window = H, 1, key, R, m.scale, m.window
         w.act_f32, w.cache_f32 = self.f32, self.f32
-        self._attend(w, L, b, 1, key, R, (lambda n: min(m.window, n)) if m.window else (lambda n: n), key)
+        self.attend(w, L['tile_rows'], b, 1, key, R, (lambda n: min(m.window, n)) if m.window else (lambda n: n), key)
         # values out of the latent space: hid[:, h, :] = V_h olat[:, h, :]
         hid = e(T, H * dv, dt=act)
         ev = self._ev()
@@ -340,7 +296,7 @@ class DanalornB200(PagedLM):
         w.out, w.ld_out = ptr(att), att.stride(0)
         w.n_heads, w.n_kv, w.dim, w.vdim, w.scale, w.window = H, G, d, dv, m.scale, 0
         w.act_f32, w.cache_f32 = self.f32, self.f32
-        self._attend(w, L, b, G, d, dv, lambda n: n, G * (d + dv))
+        self.attend(w, L['tile_rows'], b, G, d, dv, lambda n: n, G * (d + dv))
         y = e(T, W)
         self.linear(att, L['out_w'], y, nxt=L.get('up'))
         return y

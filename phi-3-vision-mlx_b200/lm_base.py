@@ -1,12 +1,13 @@
 """What the engine models (decoders with an fp32 residual stream that run a ragged token batch against the shared page pool) have in
-common: the description of a step, the choice of the matrix-product kernel, the grouped expert products and the key-slice cost model
-of the decode attention. A design (tagenex.py, tapalix.py, dugalix.py, danalorn.py) owns its weights and the order of its kernels; it has no cache and no loop
-of its own.
+common: the description of a step, the choice of the matrix-product kernel, the grouped expert products, the attention launches of a
+step and the key-slice cost model of the decode attention. A design (tagenex.py, tapalix.py, dugalix.py, danalorn.py, lupusun.py) owns
+its weights and the order of its kernels; it has no cache and no loop of its own.
 
 Matrix products. Dense bf16 products with K % 8 == 0 run on the tcgen05 GEMM (p3_gemm); batches of at most 16 tokens on the
 weight-streaming kernel (p3_gemm_skinny); everything else (fp32 = true 32-bit on the FMA pipes, grouped expert products, products
 per attention head over column blocks, odd shapes) on p3_gemm_any.
 """
+import ctypes as C
 import os
 import torch
 from . import _lib
@@ -126,6 +127,54 @@ class PagedLM:
             a.gate, a.ld_gate = ptr(gate), gate.stride(0)
         call_struct('p3_gemm_any', a, _stream())
         return out
+
+    def stacked_rows(self, parts):
+        """projection matrices over one input as one matrix in the compute type, padded with zero rows to a multiple of 16 (small
+        batches keep the weight-streaming kernel)"""
+        n = sum(p.shape[0] for p in parts)
+        if n % 16:
+            parts = parts + [torch.zeros(-n % 16, parts[0].shape[1], dtype=parts[0].dtype, device=parts[0].device)]
+        return torch.cat(parts, 0).to(self.dev, self.dtype).contiguous()
+
+    # ------------------------------------------------------------------ attention over the page pool
+    def attention_tile_rows(self, H, G, key, val, v_ld):
+        """query rows per prefill tile that the attention launch takes for these sizes (64: its tensor-core kernels); asked of the
+        library itself so that the engine's tiles and the kernel's choice cannot disagree"""
+        a = _lib.AttnWindowArgs()
+        a.q = a.out = a.k_pool = a.v_pool = a.block_table = a.tiles = 256              # aligned stand-ins: nothing is launched
+        a.ld_q, a.ld_out, a.n_heads, a.n_kv, a.dim, a.vdim, a.v_ld = H * key, H * val, H, G, key, val, v_ld
+        a.act_f32 = a.cache_f32 = self.f32
+        return int(_lib.lib().p3_attn_window_tile_rows(C.byref(a)))
+
+    def attend(self, w, tile_rows, b, G, key, val, span_of, kv_bytes, pf_span=None):
+        """the prefill tiles and the single-token requests of the step through p3_attn_window_*; span_of(n) = most keys a query at
+        position n - 1 sees, pf_span = mean keys per query of a prompt (accounting only), kv_bytes = cache numbers of one token"""
+        st, H = _stream(), w.n_heads
+        esz = 4 if self.f32 else 2
+        if b.n_pf:
+            w.tiles, w.n_tiles = ptr(b.pf_tiles), b.n_pf
+            ev = self._ev()
+            call_struct('p3_attn_window_prefill', w, st)
+            if pf_span is None:
+                pf_span = span_of(b.max_pos + 1) if w.window else (b.max_pos + 1) // 2
+            self._ev(ev, 'attn_prefill', 2 * (b.T - b.n_dec) * H * pf_span * (key + val), 0)
+        if b.n_dec:
+            w.tiles, w.n_tiles = ptr(b.dec_tiles), b.n_dec
+            span = span_of(b.max_pos + 1)
+            if tile_rows == 64:
+                if G == 1 and H > 1:
+                    # one shared K/V head: a request is one CTA per slice (two when the values take two column blocks)
+                    w.n_splits = _page_slices(b.n_dec * (-(-val // 128) if key > 128 else 1), 2 * -(-span // 128) + 1, merge=0.4)
+                else:
+                    w.n_splits = _page_slices(b.n_dec * G, 2 * -(-span // 128) + 1)
+            else:
+                # one key per lane: enough CTAs for eight per SM, at least 128 keys (one pass of a CTA) per slice
+                w.n_splits = max(1, min(-(-8 * 148 // (b.n_dec * G)), -(-span // 128)))
+            ws = torch.empty(b.n_dec * H * w.n_splits * (val + 2), dtype=torch.float32, device=self.dev) if w.n_splits > 1 else None
+            w.ws = ptr(ws)
+            ev = self._ev()
+            call_struct('p3_attn_window_decode', w, st)
+            self._ev(ev, 'attn_decode', 2 * b.n_dec * H * span * (key + val), b.n_dec * span * kv_bytes * esz)
 
     # ------------------------------------------------------------------ mixture of experts behind a router
     def experts(self, gu_w, down_w, f, xa, y, T, ids, wts, glu, n_sorted=None, combine=None):

@@ -118,9 +118,21 @@ def _danalorn_build(cfg, weights, device='cuda', dtype=None, **kw):
     return DanalornB200(cfg, weights, device=device, dtype=dtype or torch.bfloat16)
 
 
+def _lupusun_config(d):
+    from .configs import LupusunConfig
+    return LupusunConfig(d)
+
+
+def _lupusun_build(cfg, weights, device='cuda', dtype=None, **kw):
+    import torch
+    from .lupusun import LupusunB200
+    return LupusunB200(cfg, weights, device=device, dtype=dtype or torch.bfloat16)
+
+
 register('Phi3ForCausalLM', _phi3_config, _phi3_build, 'batch')
 register('Phi3VForCausalLM', _phi3_config, _phi3_build, 'batch')
 register('Tagenex', _tagenex_config, _tagenex_build, 'paged')
 register('Tapalix', _tapalix_config, _tapalix_build, 'paged')
 register('Dugalix', _dugalix_config, _dugalix_build, 'paged')
 register('Danalorn', _danalorn_config, _danalorn_build, 'paged')
+register('Lupusun', _lupusun_config, _lupusun_build, 'paged')

@@ -363,3 +363,56 @@ def random_danalorn_weights(cfg, seed=0, device='cpu'):
             t = rn(shape) / shape[-1] ** 0.5
         w[name] = t.to(torch.bfloat16)
     return w
+
+
+def lupusun_tensor_shapes(cfg):
+    """name -> shape of every tensor of a Lupusun checkpoint; cfg = the config.json dict"""
+    W, V = cfg['width'], cfg['vocab']
+    out = {'embed': (V, W), 'embed.norm': (W,)}
+    for i, lc in enumerate(cfg['layers']):
+        p, m = f'l{i}.', lc['mixer']
+        a = p + 'mix.'
+        H, d = m['heads'], m['dim']
+        G, dv = m.get('kv_heads', H), m.get('vdim', d)
+        out[p + 'norm1'] = (W,)
+        if lc['type'] == 'delta':
+            out.update({a + 'q': (G * d, W), a + 'k': (G * d, W), a + 'v': (H * dv, W), a + 'q.conv': (G * d, m['conv']),
+                        a + 'k.conv': (G * d, m['conv']), a + 'v.conv': (H * dv, m['conv']), a + 'b': (H, W), a + 'a': (H, W),
+                        a + 'A_log': (H,), a + 'dt_bias': (H,), a + 'norm': (dv,), a + 'g': (H * dv, W), a + 'o': (W, H * dv)})
+        elif lc['type'] == 'attention':
+            out.update({a + 'q': (H * d, W), a + 'q.b': (H * d,), a + 'k': (G * d, W), a + 'k.b': (G * d,), a + 'v': (G * dv, W),
+                        a + 'v.b': (G * dv,), a + 'sink': (H,), a + 'o': (W, H * dv)})
+        else:
+            raise NotImplementedError(lc['type'])
+        f = lc.get('mlp')
+        if f is not None:
+            out.update({p + 'norm2': (W,), p + 'mlp.gate': (f['ff'], W), p + 'mlp.up': (f['ff'], W), p + 'mlp.down': (W, f['ff'])})
+    out.update({'final.norm': (W,), 'head': (V, W)})
+    return out
+
+
+def random_lupusun_weights(cfg, seed=0, device='cpu'):
+    """Seeded bf16 tensors for a Lupusun config dict: matrices N(0, 1/fan_in), embedding of unit spread, norm gains around one, biases
+    0.3 N, sinks N(0, 1), convolution taps of spread 0.6; the decays' logarithms and offsets are spread so that heads remember from a
+    few tokens to hundreds."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    rn = lambda s: torch.randn(s, generator=g, device=device, dtype=torch.float32)
+    w = {}
+    for name, shape in lupusun_tensor_shapes(cfg).items():
+        leaf = name.split('.', 1)[1] if name.startswith('l') and name[1].isdigit() else name
+        if leaf == 'mix.dt_bias':
+            t = -2.5 + 1.5 * rn(shape)
+        elif leaf == 'mix.A_log':
+            t = 0.5 * rn(shape)
+        elif leaf.endswith('.conv'):
+            t = 0.6 * rn(shape)
+        elif leaf.endswith(('q.b', 'k.b', 'v.b')):
+            t = 0.3 * rn(shape)
+        elif leaf in ('embed', 'mix.sink'):
+            t = rn(shape)
+        elif 'norm' in leaf.rsplit('.', 1)[-1]:
+            t = 1.0 + 0.1 * rn(shape)
+        else:
+            t = rn(shape) / shape[-1] ** 0.5
+        w[name] = t.to(torch.bfloat16)
+    return w
