@@ -830,6 +830,67 @@ def run_danalorn(args):
           'steps': args.steps, 'warmup': max(3, args.warmup), 'peaks': {'hbm_gbs': hbm, 'bf16_tflops': tf}, 'sizes': out})
 
 
+# ------------------------------------------------------------------------------------------------ --arch lupusun
+def _lupusun_cfg(width, heads, kv, dim, chunk, dh, dkv, ddim, dvdim, ff, layers, vocab):
+    att = {'type': 'attention',
+           'mixer': {'heads': heads, 'kv_heads': kv, 'dim': dim, 'vdim': dim, 'scale': dim ** -0.5, 'mask': {'size': chunk},
+                     'rot': {'base': 500000.0, 'dims': dim, 'scaling': {'factor': 4.0, 'original': 4096, 'fast': 32.0, 'slow': 1.0}}}}
+    delta = {'type': 'delta', 'mixer': {'heads': dh, 'kv_heads': dkv, 'dim': ddim, 'vdim': dvdim, 'conv': 4}}
+    order = [delta, att, delta, att]
+    return {'architecture': 'Lupusun', 'vocab': vocab, 'width': width, 'norm': {'eps': 1e-5}, 'residual_mult': 0.9,
+            'layers': [dict(order[i % 4], mlp={'kind': 'dense', 'ff': ff}) for i in range(layers)]}
+
+
+def run_lupusun(args):
+    """Throughput of the Lupusun design on the continuous-batching engine at layer sizes of a real model (random weights, bf16
+    serving mode), beside Danalorn, the closest existing model (same engine, page pool with state rows, product kernels, attention
+    kernels, a recurrent scan of the same layout with the same head norm and gate behind it), at equal width, depth, attention shape,
+    recurrent state shape and feed-forward size. One JSON line: per size the prefill and decode tok/s of both and, per kernel
+    family, time and achieved FLOP/s (prefill) or bytes/s (decode) against the measured peaks."""
+    import torch
+    import phi3_b200  # noqa: F401
+    from phi3_b200 import weights
+    from phi3_b200.danalorn import DanalornB200
+    from phi3_b200.lupusun import LupusunB200
+    hbm, _ = peaks()
+    tf = json.load(open(os.path.join(ROOT, 'MEASURED_PEAKS.json'))).get('bf16_tflops', 1590.0) if os.path.exists(
+        os.path.join(ROOT, 'MEASURED_PEAKS.json')) else 1590.0
+    dev = torch.device('cuda:0')
+    sizes = [dict(name='w2048_h16x128_kv4_chunk1024_d8x128x256_ff8192_L4', width=2048, heads=16, kv=4, dim=128, chunk=1024, dh=8, dkv=8,
+                  ddim=128, dvdim=256, ff=8192, layers=4),
+             dict(name='w2048_h16x128_kv4_chunk1024_d8x128x256_ff8192_L4_b16', width=2048, heads=16, kv=4, dim=128, chunk=1024, dh=8, dkv=8,
+                  ddim=128, dvdim=256, ff=8192, layers=4, batch=16),
+             dict(name='w3072_h32x64_kv8_chunk512_d12/6x64x256_ff8192_L4', width=3072, heads=32, kv=8, dim=64, chunk=512, dh=12, dkv=6,
+                  ddim=64, dvdim=256, ff=8192, layers=4)]
+    if getattr(args, 'sizes', None):
+        sizes = [sz for i, sz in enumerate(sizes) if str(i) in args.sizes.split(',')]
+    vocab, L, CTX_D, NEW_D = 32064, 2048, 2048, 32
+    out = []
+    for sz in sizes:
+        B = sz.get('batch', 4)
+        cfg = _lupusun_cfg(sz['width'], sz['heads'], sz['kv'], sz['dim'], sz['chunk'], sz['dh'], sz['dkv'], sz['ddim'], sz['dvdim'],
+                           sz['ff'], sz['layers'], vocab)
+        m = LupusunB200(cfg, weights.random_lupusun_weights(cfg, 0, device=dev), dtype=torch.bfloat16)
+        _, nums = _engine_model_numbers(m, B, L, CTX_D, NEW_D, vocab, args, hbm, tf)
+        row = dict(size=sz['name'], batch=B, prompt=L, lupusun=nums)
+        del m
+        torch.cuda.empty_cache()
+        # Danalorn at equal size: biased attention of the same shape (causal over the whole context), gated linear attention of the
+        # recurrent state's shape, a relu^2 unit of the same inner size
+        att = {'type': 'attention', 'mixer': {'heads': sz['heads'], 'kv_heads': sz['kv'], 'dim': sz['dim'], 'vdim': sz['dim'],
+                                              'scale': sz['dim'] ** -0.5, 'q_temp': {'coef': 0.25, 'every': 128}}}
+        gla = {'type': 'gla', 'mixer': {'heads': sz['dh'], 'dim': sz['ddim'], 'vdim': sz['dvdim'], 'tau': 8.0}}
+        dcfg = {'architecture': 'Danalorn', 'vocab': vocab, 'width': sz['width'], 'norm': {'eps': 1e-5}, 'embedding': {'scale': 1.0},
+                'layers': [dict(att if i % 2 else gla, mlp={'kind': 'dense', 'ff': sz['ff']}) for i in range(sz['layers'])]}
+        dm = DanalornB200(dcfg, weights.random_danalorn_weights(dcfg, 0, device=dev), dtype=torch.bfloat16)
+        _, row['danalorn_equal_size'] = _engine_model_numbers(dm, B, L, CTX_D, NEW_D, vocab, args, hbm, tf)
+        del dm
+        torch.cuda.empty_cache()
+        out.append(row)
+    _emit({"metric": "lupusun_prefill_decode_tok_per_s", 'arch': 'lupusun', 'dtype': 'bf16', 'data': 'synthetic', 'n_gpus': 1,
+          'steps': args.steps, 'warmup': max(3, args.warmup), 'peaks': {'hbm_gbs': hbm, 'bf16_tflops': tf}, 'sizes': out})
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument('--gpus', type=int, default=1)
@@ -837,10 +898,10 @@ def main():
     ap.add_argument('--warmup', type=int, default=3)
     ap.add_argument('--impl', default='b200', choices=['b200', 'reference'])
     ap.add_argument('--no-cpu-baseline', action='store_true')
-    ap.add_argument('--arch', default='phi3', choices=['phi3', 'tagenex', 'tapalix', 'dugalix', 'danalorn'],
-                    help='phi3: the headline workload (default); tagenex / tapalix / dugalix / danalorn: prefill / decode throughput of '
+    ap.add_argument('--arch', default='phi3', choices=['phi3', 'tagenex', 'tapalix', 'dugalix', 'danalorn', 'lupusun'],
+                    help='phi3: the headline workload (default); tagenex / tapalix / dugalix / danalorn / lupusun: prefill / decode throughput of '
                          'that design on the continuous-batching engine, beside the closest existing model at equal size')
-    ap.add_argument('--sizes', default='', help='with --arch dugalix / danalorn: indices of the sizes to run, with commas (default: all)')
+    ap.add_argument('--sizes', default='', help='with --arch dugalix / danalorn / lupusun: indices of the sizes to run, with commas (default: all)')
     args = ap.parse_args()
     if not (args.gpus > 1 and int(os.environ.get('WORLD_SIZE', 1)) == 1):      # the self-launching parent just relays its child
         _claim_stdout()
@@ -854,6 +915,8 @@ def main():
         return run_dugalix(args)
     if args.arch == 'danalorn':
         return run_danalorn(args)
+    if args.arch == 'lupusun':
+        return run_lupusun(args)
     world = int(os.environ.get('WORLD_SIZE', 1))
     if args.gpus > 1 and world == 1:
         # convenience: self-launch under torchrun when called directly with --gpus N
