@@ -29,6 +29,17 @@ __device__ __forceinline__ float block_sum(float v, float* sh) {
     return t;
 }
 
+// two sums at once (sh: 64 floats)
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* sh) {
+    a = warp_sum(a); b = warp_sum(b);
+    const int w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    if ((threadIdx.x & 31) == 0) { sh[2 * w] = a; sh[2 * w + 1] = b; }
+    __syncthreads();
+    float2 t = make_float2(0.f, 0.f);
+    for (int i = 0; i < nw; i++) { t.x += sh[2 * i]; t.y += sh[2 * i + 1]; }
+    return t;
+}
+
 // ---------------------------------------------------------------- embedding -> fp32 residual (+ activation copy)
 // Row kernels below keep up to RPT elements per thread in registers: all loads of a pass are issued before the first use, so a
 // row of a small batch costs a few memory round trips instead of one per loop iteration.
@@ -971,19 +982,22 @@ template <int VEC, typename AT> __device__ __forceinline__ void row_store(AT* p,
 }
 
 // ---------------------------------------------------------------- embedding row under a norm (+ copy, + the first layer's norm of it)
+// The second norm's sum of squares is formed beside the first one's, without the common factor r of the normed row: one reduction.
 template <typename AT, int VEC>
 __global__ void embed_norm_rows_kernel(const bf16* __restrict__ table, const int32_t* __restrict__ ids, const float* __restrict__ gain,
                                        float* __restrict__ x, float* __restrict__ copy, const float* __restrict__ gpre, AT* __restrict__ h,
                                        int W, int vocab, float eps) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
     pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
-    __shared__ float sh[32];
+    __shared__ float sh[64];
     const int64_t t = blockIdx.x;
     int id = ids[t];
     if (id < 0 || id >= vocab) id = 0;
     const bf16* src = table + (size_t)id * W;
     const int nt = blockDim.x;
-    float v[RPT], gv[RPT];
+    float v[RPT], gv[RPT], gp[RPT];
+    row_load<VEC>(gain, W, gv);
+    if (gpre) row_load<VEC>(gpre, W, gp);
 #pragma unroll
     for (int k = 0; k < RPT; k += VEC) {
         const int i = row_at<VEC>(k);
@@ -993,32 +1007,31 @@ __global__ void embed_norm_rows_kernel(const bf16* __restrict__ table, const int
             v[k] = lo.x; v[k + 1] = lo.y; v[k + 2] = hi.x; v[k + 3] = hi.y;
         } else v[k] = i < W ? __bfloat162float(src[i]) : 0.f;
     }
-    row_load<VEC>(gain, W, gv);
-    float ss = 0.f;
+    float ss = 0.f, s2 = 0.f;
 #pragma unroll
-    for (int k = 0; k < RPT; k++) ss = fmaf(v[k], v[k], ss);
-    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) { const float u = __bfloat162float(src[i]); ss = fmaf(u, u, ss); }
-    ss = block_sum(ss, sh);
-    const float r = 1.0f / sqrtf(ss / (float)W + eps);
-    float s2 = 0.f;
+    for (int k = 0; k < RPT; k++) { ss = fmaf(v[k], v[k], ss); v[k] *= gv[k]; s2 = fmaf(v[k], v[k], s2); }
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) {
+        const float u = __bfloat162float(src[i]), ug = u * gain[i];
+        ss = fmaf(u, u, ss); s2 = fmaf(ug, ug, s2);
+    }
+    const float2 sum = block_sum2(ss, s2, sh);
+    const float r = 1.0f / sqrtf(sum.x / (float)W + eps);
 #pragma unroll
-    for (int k = 0; k < RPT; k++) { v[k] = v[k] * r * gv[k]; s2 = fmaf(v[k], v[k], s2); }
+    for (int k = 0; k < RPT; k++) v[k] *= r;
     row_store<VEC>(x + (size_t)t * W, W, v);
     if (copy) row_store<VEC>(copy + (size_t)t * W, W, v);
+    const float r2 = 1.0f / sqrtf(sum.y * r * r / (float)W + eps);
+    if (gpre) {
+#pragma unroll
+        for (int k = 0; k < RPT; k++) v[k] = v[k] * r2 * gp[k];
+        row_store<VEC>(h + (size_t)t * W, W, v);
+    }
     for (int i = threadIdx.x + RPT * nt; i < W; i += nt) {
-        const float u = __bfloat162float(src[i]) * r * gain[i];
+        const float u = __bfloat162float(src[i]) * gain[i] * r;
         x[(size_t)t * W + i] = u;
         if (copy) copy[(size_t)t * W + i] = u;
-        s2 = fmaf(u, u, s2);
+        if (gpre) stv(h + (size_t)t * W + i, u * r2 * gpre[i]);
     }
-    if (!gpre) return;
-    row_load<VEC>(gpre, W, gv);
-    s2 = block_sum(s2, sh);
-    const float r2 = 1.0f / sqrtf(s2 / (float)W + eps);
-#pragma unroll
-    for (int k = 0; k < RPT; k++) v[k] = v[k] * r2 * gv[k];
-    row_store<VEC>(h + (size_t)t * W, W, v);
-    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) stv(h + (size_t)t * W + i, x[(size_t)t * W + i] * r2 * gpre[i]);   // this thread's own write
 }
 
 // ---------------------------------------------------------------- x += mult * y (+ add) ; h = rms_norm(x) * gain
@@ -1383,11 +1396,17 @@ extern "C" int p3_distance_linear_table(const float* slope, float* pen, int H, i
     return 0;
 }
 
+// threads of a CTA whose registers hold a row of W numbers, RPT each (up to W = 8192; longer rows go through memory)
+static int row_threads(int W) {
+    const int th = (W + RPT * 32 - 1) / (RPT * 32) * 32;
+    return th < 128 ? 128 : th > 1024 ? 1024 : th;
+}
+
 extern "C" int p3_embed_norm_rows_f32(const void* table, const int32_t* ids, const float* gain, float* x, float* copy, const float* gain_pre,
                                       void* h, int act_f32, int64_t T, int W, int vocab, float eps, cudaStream_t st) {
     P3_CHECK_ARG(table && ids && gain && x && (!gain_pre || h), "embed_norm_rows_f32: null argument");
     if (T == 0) return 0;
-    const int th = W > 4096 ? 1024 : W > 2048 ? 512 : W >= 1024 ? 256 : 128;     // the row fits the threads' registers up to W = 8192
+    const int th = row_threads(W);
     const bool vec = W % 4 == 0 && (((uintptr_t)gain | (uintptr_t)x | (uintptr_t)copy | (uintptr_t)gain_pre | (uintptr_t)h) & 15) == 0 &&
                      ((uintptr_t)table & 7) == 0;
 #define GO(AT, V) p3_launch_pdl(embed_norm_rows_kernel<AT, V>, dim3((unsigned)T), dim3(th), (size_t)(0), st, (const bf16*)table, ids, gain, x, copy, gain_pre, (AT*)h, W, vocab, eps)
@@ -1402,7 +1421,7 @@ extern "C" int p3_residual_rmsnorm(float* x, const float* y, int64_t ldy, float 
                                    const float* gain, void* h, int act_f32, int64_t R, int W, float eps, cudaStream_t st) {
     P3_CHECK_ARG(x && W >= 1 && (!gain || h), "residual_rmsnorm: null argument");
     if (R == 0) return 0;
-    const int th = W > 4096 ? 1024 : W > 2048 ? 512 : W >= 1024 ? 256 : 128;
+    const int th = row_threads(W);
     const bool vec = W % 4 == 0 && (!y || ldy % 4 == 0) &&
                      (((uintptr_t)x | (uintptr_t)y | (uintptr_t)add | (uintptr_t)gain | (uintptr_t)h) & 15) == 0;
 #define GO(AT, V) p3_launch_pdl(residual_rmsnorm_kernel<AT, V>, dim3((unsigned)R), dim3(th), (size_t)(0), st, x, y, ldy, mult, add, rows, gain, (AT*)h, W, eps)
