@@ -10,10 +10,10 @@ differ between layers (`layout` = [(kv_heads, key size, value size), ...]; a lay
 numbers, so a masked slot can never poison a weighted sum. The block table lives on the device; the host keeps a mirror and
 uploads the rows that changed before a step.
 
-Recurrent state. A model whose layers carry a state from token to token (a token shift, a matrix memory, the last token) names the fp32 numbers
-each of its state buffers needs per sequence (`state_layout` = [numbers per slot, ...]); the pool allocates them once as
-[slots][numbers] and a sequence's state lives in the row of its slot. Nothing is cleared when a slot changes hands: the kernels
-start a sequence whose first token has position 0 from the zero state whatever the row holds.
+Recurrent state. A model whose layers carry a state from token to token (a token shift, a matrix memory, the last token, the last
+inputs of a convolution) names the fp32 numbers each of its state buffers needs per sequence (`state_layout` = [numbers per slot,
+...]); the pool allocates them once as [slots][numbers] and a sequence's state lives in the row of its slot. Nothing is cleared when a
+slot changes hands: the kernels start a sequence whose first token has position 0 from the zero state whatever the row holds.
 """
 import torch
 
