@@ -458,7 +458,7 @@ int p3_latent_post(const p3_latent_post_args* args, cudaStream_t st);
 
 /* out (act) [R, F] = silu(g[r][c]) * u[r][c]; g and u fp32 with the common row pitch ld */
 int p3_glu_silu(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, cudaStream_t st);
-/* the same with another activation in front of the product: act 0 = silu, 1 = relu (max(g, 0) * u) */
+/* the same with another activation in front of the product: act 0 = silu, 1 = relu (max(g, 0) * u), 2 = the tanh form of gelu */
 int p3_glu_act(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, int act, cudaStream_t st);
 
 /* router with sigmoid scores: z = Wr x (fp32; or logits fp32 [T, ld_logits] when an earlier product already formed them with fp32
@@ -497,7 +497,10 @@ int p3_token_shift(const float* h, const float* shift, float* state, const int32
  * numbers of every query and key head turn by position * freq[i] (number i paired with i + rot_n / 2, freq fp32 [rot_n / 2]), the
  * rest passes; q -> q_out (act), k -> K pool, v -> V pool. v_off < 0: there is no value projection, the value of a token is its key
  * BEFORE the rotation (vdim == dim). rot_mag: factor on cos and sin (0 is read as 1). unit_norm != 0: every query and key head is then
- * divided by its root mean square, sqrt(mean over dim of the squares + eps), after the rotation. */
+ * divided by its root mean square, sqrt(mean over dim of the squares + eps), after the rotation. pair_mode: rotation pairs, 0 = number i
+ * with i + rot_n / 2, 1 = neighbours 2i and 2i + 1 (freq[i] each). n_act > 0: the n_act numbers from act_cols on in every row (an address
+ * inside proj's first row, same pitch; columns outside q, k and v) pass silu in place: the inputs of a recurrent mixer that shares the
+ * projection. */
 typedef struct {
     const float* proj; int64_t ld_proj; int32_t q_off, k_off, v_off;
     const float* bias;
@@ -507,6 +510,7 @@ typedef struct {
     const int32_t* tok_slot; const int32_t* tok_pos; int32_t T;
     int32_t act_f32, cache_f32;
     float rot_mag; int32_t unit_norm; float eps;
+    int32_t pair_mode; float* act_cols; int32_t n_act;
 } p3_qkv_rope_post_args;
 int p3_qkv_rope_post(const p3_qkv_rope_post_args* args, cudaStream_t st);
 
@@ -612,12 +616,13 @@ int p3_residual_rmsnorm(float* x, const float* y, int64_t ldy, float mult, const
 
 /* Short causal convolutions over time, one per channel, silu, and unit length per head; and the gates of a gated delta rule.
  * Inputs are the columns [c_off, c_off + C) of proj (fp32 [n_rows, ld_proj]), C = n_unit * dim + n_plain:
- *   z_t[c] = silu(sum_j w[j][c] x_(t - (taps - 1) + j)[c])   (w fp32 [taps][C]; zeros before the start of a sequence)
+ *   z_t[c] = silu(bias[c] + sum_j w[j][c] x_(t - (taps - 1) + j)[c])   (w fp32 [taps][C], bias fp32 [C] or NULL; zeros before the start
+ *   of a sequence)
  * The leading n_unit heads of dim (<= 512) channels are divided by sqrt(sum of squares + unit_eps), the first n_scaled of them also
  * multiplied by `scale`. out fp32 [n_rows, ld_out], column c. Inputs of earlier steps come from conv_state fp32
- * [slots][taps - 1][C] (the last taps - 1 inputs in order of time), which this call only READS: p3_delta_scan advances it.
- * gates (fp32 [n_rows][n_gates][2] or NULL): {decay, beta} of every head, decay = exp(-exp(a_log) softplus(proj[a_off + h] + dt_bias)),
- * beta = sigmoid(proj[b_off + h]). */
+ * [slots][taps - 1][C] (the last taps - 1 inputs in order of time), which this call only READS: the scan behind it advances it.
+ * gates (fp32 [n_rows][n_gates][2] or NULL): with step = softplus(proj[a_off + h] + dt_bias) and decay = exp(-exp(a_log) step) of every
+ * head, gate_mode 0: {decay, sigmoid(proj[b_off + h])}, 1: {decay, step}. */
 typedef struct {
     const float* proj; int64_t ld_proj; int32_t c_off;
     int32_t n_unit, dim, n_scaled, n_plain;
@@ -626,6 +631,7 @@ typedef struct {
     const int32_t* seqs; const int32_t* slot_seq; const int32_t* tok_slot; int32_t n_rows;
     float* out; int64_t ld_out;
     int32_t a_off, b_off, n_gates; const float* a_log; const float* dt_bias; float* gates;
+    const float* bias; int32_t gate_mode;
 } p3_short_conv_args;
 int p3_short_conv(const p3_short_conv_args* args, cudaStream_t st);
 
@@ -643,9 +649,37 @@ typedef struct {
     float* state; const int32_t* seqs; int32_t n_seqs;
     float* out; int64_t ld_out; int32_t rs_force;
     const float* conv_in; int64_t ld_conv_in; int32_t channels, taps; float* conv_state;
+    const float* decay; const float* skip;     /* p3_decay_scan only */
 } p3_delta_scan_args;
 int64_t p3_delta_state_floats(int n_heads, int dim, int vdim);
 int p3_delta_scan(const p3_delta_scan_args* args, cudaStream_t st);
+
+
+/* ---- parts of decoders with several residual streams per token, a mixer of rotated attention and a linear memory with fixed decays side
+ * by side, and a state-space mixer (Gugezen and designs built from these parts) */
+
+/* The memory of p3_delta_scan without the correction at the key, same state:
+ *   S <- decay S + step k v^T,  y = S^T q + skip v
+ * decay and step from gates fp32 [T][n_heads][2], or (gates NULL) decay fp32 [n_heads] and step = 1; skip fp32 [n_heads] or NULL. */
+int p3_decay_scan(const p3_delta_scan_args* args, cudaStream_t st);
+
+/* Rows of parts * n numbers, every part normed on its own. With f = the gate's factor (sigmoid(g), or g sigmoid(g) with gate_silu; gate
+ * fp32 logits [T, ld_gate] or NULL: 1), gain fp32 [parts * n]:
+ *   gate_first: v = y f, out = v / sqrt(mean(v^2) + eps) * gain * scale;  else: out = y / sqrt(mean(y^2) + eps) * gain * f * scale */
+int p3_part_norm_gate(const float* y, int64_t ldy, int parts, int n, const float* gain, const float* gate, int64_t ld_gate, int gate_silu,
+                      int gate_first, float scale, float eps, void* out, int64_t ldo, int out_f32, int64_t T, cudaStream_t st);
+
+/* Residual streams (hyper-connections), x fp32 [T][S][W], S <= 16, t = rows ? rows[r] : r:
+ *   with y (fp32 [T, ldy]): X_to <- sum_from mix[from][to] X_from + out_w[to] y, all streams from the old ones (kept in registers only when
+ *   `rows` is given); with gain: h[r] (activation type) = u / sqrt(mean(u^2) + eps) * gain, u = sum_s in_w[s] X_s of the new streams */
+int p3_streams_rmsnorm(float* x, int S, const float* y, int64_t ldy, const float* mix, const float* out_w, const float* in_w,
+                       const int32_t* rows, const float* gain, void* h, int act_f32, int64_t R, int W, float eps, cudaStream_t st);
+/* X_s = table[ids[t]] * scale for every s (bf16 table), and h as above */
+int p3_embed_streams(const void* table, const int32_t* ids, float scale, float* x, int S, const float* in_w, const float* gain, void* h,
+                     int act_f32, int64_t T, int W, int vocab, float eps, cudaStream_t st);
+
+/* out (act) [R, F] = act(u), u fp32 with row pitch ld; act 0 = gelu (erf), 1 = its tanh form: a unit without a gate */
+int p3_unit_act(const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, int act, cudaStream_t st);
 
 #ifdef __cplusplus
 }

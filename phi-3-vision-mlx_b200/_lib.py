@@ -93,11 +93,17 @@ _SIGS = {
     'p3_embed_norm_rows_f32': [_p, _p, _p, _p, _p, _p, _p, _i, _l, _i, _i, _f, _p],
     'p3_residual_rmsnorm': [_p, _p, _l, _f, _p, _p, _p, _p, _i, _l, _i, _f, _p],
     'p3_glu_act': [_p, _p, _l, _p, _l, _i, _l, _i, _i, _p],
+    # several residual streams per token, norm in equal parts with a gate, unit without a gate (csrc/seq_ops.cu, csrc/recurrent.cu)
+    'p3_embed_streams': [_p, _p, _f, _p, _i, _p, _p, _p, _i, _l, _i, _i, _f, _p],
+    'p3_streams_rmsnorm': [_p, _i, _p, _l, _p, _p, _p, _p, _p, _p, _i, _l, _i, _f, _p],
+    'p3_part_norm_gate': [_p, _l, _i, _i, _p, _p, _l, _i, _i, _f, _f, _p, _l, _i, _l, _p],
+    'p3_unit_act': [_p, _l, _p, _l, _i, _l, _i, _i, _p],
 }
-GLU_SILU, GLU_RELU = 0, 1                                                 # activations of p3_glu_act
+UNIT_GELU, UNIT_GELU_TANH = 0, 1                                          # activations of p3_unit_act
+GLU_SILU, GLU_RELU, GLU_GELU_TANH = 0, 1, 2                                                 # activations of p3_glu_act
 ROUTER_SOFTMAX, ROUTER_GROUP_MAX, ROUTER_PLAIN_WEIGHTS = 1, 2, 4          # mode bits of p3_router_groups
 _STRUCT_ENTRIES = ['p3_gemm_any', 'p3_qkv_post', 'p3_attn_window_prefill', 'p3_attn_window_decode', 'p3_latent_post',
-                   'p3_qkv_rope_post', 'p3_matrix_memory_scan', 'p3_gla_scan', 'p3_short_conv', 'p3_delta_scan']
+                   'p3_qkv_rope_post', 'p3_matrix_memory_scan', 'p3_gla_scan', 'p3_short_conv', 'p3_delta_scan', 'p3_decay_scan']
 ATTN_WINDOW_MMA = os.environ.get('P3_ATTN_WINDOW_MMA', '1') != '0'
 
 _lib = None
@@ -272,7 +278,8 @@ class QkvRopePostArgs(C.Structure):
                 ('freq', _p), ('q_out', _p), ('ld_q', _l),
                 ('k_pool', _p), ('v_pool', _p), ('block_table', _p), ('bt_stride', C.c_int32),
                 ('tok_slot', _p), ('tok_pos', _p), ('T', C.c_int32), ('act_f32', C.c_int32), ('cache_f32', C.c_int32),
-                ('rot_mag', C.c_float), ('unit_norm', C.c_int32), ('eps', C.c_float)]
+                ('rot_mag', C.c_float), ('unit_norm', C.c_int32), ('eps', C.c_float),
+                ('pair_mode', C.c_int32), ('act_cols', _p), ('n_act', C.c_int32)]
 
 
 class MatrixMemoryArgs(C.Structure):
@@ -298,7 +305,8 @@ class ShortConvArgs(C.Structure):
                 ('n_unit', C.c_int32), ('dim', C.c_int32), ('n_scaled', C.c_int32), ('n_plain', C.c_int32),
                 ('w', _p), ('taps', C.c_int32), ('conv_state', _p), ('scale', C.c_float), ('unit_eps', C.c_float),
                 ('seqs', _p), ('slot_seq', _p), ('tok_slot', _p), ('n_rows', C.c_int32), ('out', _p), ('ld_out', _l),
-                ('a_off', C.c_int32), ('b_off', C.c_int32), ('n_gates', C.c_int32), ('a_log', _p), ('dt_bias', _p), ('gates', _p)]
+                ('a_off', C.c_int32), ('b_off', C.c_int32), ('n_gates', C.c_int32), ('a_log', _p), ('dt_bias', _p), ('gates', _p),
+                ('bias', _p), ('gate_mode', C.c_int32)]
 
 
 class DeltaScanArgs(C.Structure):
@@ -306,4 +314,5 @@ class DeltaScanArgs(C.Structure):
     _fields_ = [('qkv', _p), ('ld_qkv', _l), ('q_off', C.c_int32), ('k_off', C.c_int32), ('v_off', C.c_int32), ('gates', _p),
                 ('n_heads', C.c_int32), ('n_kv', C.c_int32), ('dim', C.c_int32), ('vdim', C.c_int32),
                 ('state', _p), ('seqs', _p), ('n_seqs', C.c_int32), ('out', _p), ('ld_out', _l), ('rs_force', C.c_int32),
-                ('conv_in', _p), ('ld_conv_in', _l), ('channels', C.c_int32), ('taps', C.c_int32), ('conv_state', _p)]
+                ('conv_in', _p), ('ld_conv_in', _l), ('channels', C.c_int32), ('taps', C.c_int32), ('conv_state', _p),
+                ('decay', _p), ('skip', _p)]

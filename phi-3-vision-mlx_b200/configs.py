@@ -154,13 +154,13 @@ def layer_runs(loop, n):
     return SimpleNamespace(start=lo, stop=hi, times=times), [(i, i == lo) for i in order]
 
 
-def scaled_rotation(i, r, width, what):
-    """config entry {"base", "dims", "scaling": {"factor", "original", "fast", "slow"} or absent} of layer i -> namespace for
-    yarn_frequencies; `width`: how many numbers of a head may turn (the default of dims), `what`: its name in the config"""
+def scaled_rotation(i, r, width, what, keys=('factor', 'original', 'fast', 'slow')):
+    """config entry {"base", "dims", "scaling": {one number per key of `keys`} or absent} of layer i -> namespace for
+    yarn_frequencies / wavelength_frequencies; `width`: how many numbers of a head may turn (the default of dims), `what`: its name in
+    the config"""
     sc = r.get('scaling')
     rot = SimpleNamespace(base=float(r['base']), dims=int(r.get('dims', width)),
-                          scaling=None if not sc else SimpleNamespace(factor=float(sc['factor']), original=float(sc['original']),
-                                                                      fast=float(sc['fast']), slow=float(sc['slow'])))
+                          scaling=None if not sc else SimpleNamespace(**{k: float(sc[k]) for k in keys}))
     if rot.dims % 2 or not 0 < rot.dims <= width:
         raise ValueError(f'layer {i}: rot.dims must be even and at most {what}')
     return rot
@@ -590,3 +590,156 @@ def tiny_lupusun(width=96, vocab=300, layers=None, loop=(1, 3, 2), eps=1e-5, res
     if loop:
         d['loop'] = {'start': loop[0], 'stop': loop[1], 'times': loop[2]}
     return d
+
+
+# ------------------------------------------------------------------------------------------------ Gugezen
+class GugezenConfig:
+    """config.json of a Gugezen checkpoint: {"architecture": "Gugezen", "vocab", "width", "norm": {"eps"}, "embedding": {"scale"},
+    "streams", "logit_scale", "layers": [...]}. A layer entry has "type", "mixer" and "mlp":
+      type "parallel": mixer = {left: {heads, kv_heads, dim, vdim, scale, rot: {base, dims, scaling: {factor, low, high, original}}},
+                       right: {heads, dim, vdim, decay: [one factor per head]}, left_scale, right_scale}: biased attention with a rotation
+                       of neighbour pairs, a learned per-head sink and an element-wise gate, beside a linear memory with fixed decays;
+      type "mamba2":   mixer = {heads, vdim, state, groups, conv, norm_groups}: a state-space mixer;
+      mlp: null | {"kind": "dense", ff}: a gated unit with the tanh form of gelu | {"kind": "moe", expert: {ff}, router: {experts, top},
+                       shared: {ff}}: gelu units without a gate behind a softmax router, plus a shared one.
+    A layer with "weights_of": j uses the tensors of layer j (whose entry it repeats) with a cache or state of its own. Absent optional
+    keys mean: one stream, factors of one, no rotation, plain frequencies, one group, one part in the norm, no shared unit. Nothing is
+    assumed equal between layers. `sources[i]` is the layer whose tensors layer i uses."""
+    MAX_STREAMS = 16             # what the kernels take
+
+    @staticmethod
+    def _attention(i, m):
+        a = SimpleNamespace(heads=int(m['heads']), kv_heads=int(m.get('kv_heads', m['heads'])), dim=int(m['dim']),
+                            vdim=int(m.get('vdim', m['dim'])), scale=float(m['scale']), rot=None)
+        if a.heads % a.kv_heads:
+            raise ValueError(f'layer {i}: heads must be a multiple of kv_heads')
+        if a.dim > 4096 or a.vdim > 4096:
+            raise NotImplementedError(f'layer {i}: head sizes above 4096; the attention kernels take at most that')
+        r = m.get('rot')
+        if r and int(r.get('dims', a.dim)) != 0:
+            a.rot = scaled_rotation(i, r, a.dim, 'dim', ('factor', 'low', 'high', 'original'))
+        return a
+
+    def _mixer(self, i, kind, m):
+        if kind == 'parallel':
+            r = m['right']
+            mem = SimpleNamespace(heads=int(r['heads']), dim=int(r['dim']), vdim=int(r.get('vdim', r['dim'])),
+                                  decay=[float(x) for x in r['decay']])
+            if len(mem.decay) != mem.heads:
+                raise ValueError(f'layer {i}: {len(mem.decay)} decays for {mem.heads} heads')
+            if not 1 <= mem.dim <= 512:
+                raise NotImplementedError(f'layer {i}: key size {mem.dim} of the recurrence; the kernels take 1 .. 512')
+            return SimpleNamespace(kind=kind, att=self._attention(i, m['left']), mem=mem, att_scale=float(m.get('left_scale', 1.0)),
+                                   mem_scale=float(m.get('right_scale', 1.0)))
+        if kind == 'mamba2':
+            s = SimpleNamespace(kind=kind, heads=int(m['heads']), vdim=int(m['vdim']), state=int(m['state']), groups=int(m.get('groups', 1)),
+                                taps=int(m['conv']), norm_groups=int(m.get('norm_groups', 1)))
+            s.inner = s.heads * s.vdim
+            s.channels = s.inner + 2 * s.groups * s.state                    # of the convolution: x | B | C
+            if s.heads % s.groups:
+                raise ValueError(f'layer {i}: heads must be a multiple of groups')
+            if s.norm_groups < 1 or s.inner % s.norm_groups:
+                raise ValueError(f'layer {i}: norm_groups must divide heads * vdim')
+            if s.taps < 1:
+                raise ValueError(f'layer {i}: the convolution needs at least one tap')
+            if not 1 <= s.state <= 512:
+                raise NotImplementedError(f'layer {i}: state size {s.state}; the kernels take 1 .. 512')
+            return s
+        raise NotImplementedError(f'layer {i}: mixer type {kind!r} is not part of this design')
+
+    @staticmethod
+    def _ff(i, f):
+        if f is None:
+            return None
+        if f['kind'] == 'dense':
+            return SimpleNamespace(kind='dense', ff=int(f['ff']))
+        if f['kind'] == 'moe':
+            ff = SimpleNamespace(kind='moe', ff=int(f['expert']['ff']), experts=int(f['router']['experts']), top=int(f['router']['top']),
+                                 shared_ff=int((f.get('shared') or {}).get('ff', 0)))
+            if not 1 <= ff.top <= ff.experts:
+                raise ValueError(f'layer {i}: top must be in [1, experts]')
+            if ff.experts > 1024:
+                raise NotImplementedError(f'layer {i}: {ff.experts} experts; the router takes at most 1024')
+            return ff
+        raise NotImplementedError(f"layer {i}: feed-forward kind {f['kind']!r}")
+
+    def __init__(self, d):
+        self.raw = d
+        self.architecture = d.get('architecture', 'Gugezen')
+        self.architectures = [self.architecture]
+        self.vocab_size, self.width = int(d['vocab']), int(d['width'])
+        self.eps = float(d['norm']['eps'])
+        self.embed_scale = float((d.get('embedding') or {}).get('scale', 1.0))
+        ls = d.get('logit_scale')
+        self.logit_scale = 1.0 if ls is None else float(ls)
+        self.streams = int(d.get('streams') or 1)
+        if self.streams < 1:
+            raise ValueError('streams must be at least 1')
+        if self.streams > self.MAX_STREAMS:
+            raise NotImplementedError(f'{self.streams} residual streams; the kernels take at most {self.MAX_STREAMS}')
+        entries = d['layers']
+        self.sources, self.layers = [], []
+        for i, lc in enumerate(entries):
+            j, seen = i, {i}
+            while entries[j].get('weights_of') is not None:
+                j = int(entries[j]['weights_of'])
+                if not 0 <= j < len(entries) or j in seen:
+                    raise ValueError(f'layer {i}: weights_of must lead to a layer with tensors of its own')
+                seen.add(j)
+            for k in ('type', 'mixer', 'mlp'):
+                if j != i and k in lc and lc[k] != entries[j].get(k):
+                    raise ValueError(f'layer {i}: its {k} differs from that of layer {j}, whose tensors it uses')
+            self.sources.append(j)
+            self.layers.append(SimpleNamespace(mixer=self._mixer(i, entries[j].get('type'), entries[j]['mixer']),
+                                               ff=self._ff(i, entries[j].get('mlp'))))
+        self.num_hidden_layers = len(self.layers)
+
+    def kv_layout(self):
+        """per layer (kv heads, key size, value size): what the page pool allocates; a state-space layer caches nothing"""
+        return [(l.mixer.att.kv_heads, l.mixer.att.dim, l.mixer.att.vdim) if l.mixer.kind == 'parallel' else (0, 0, 0) for l in self.layers]
+
+
+def wavelength_frequencies(rot):
+    """angular frequency of every turning pair. Pair i turns by base^(-2i/dims) per position. With scaling, pairs whose wavelength is
+    shorter than original / high keep their frequency, those longer than original / low are slowed by the factor, and in between the
+    two frequencies are blended linearly in original / wavelength (the long-context scaling of Llama 3.1)."""
+    import math
+    f = [rot.base ** (-2.0 * i / rot.dims) for i in range(rot.dims // 2)]
+    sc = rot.scaling
+    if sc is None:
+        return f
+    out = []
+    for x in f:
+        wl = 2.0 * math.pi / x
+        if wl < sc.original / sc.high:
+            out.append(x)
+        elif wl > sc.original / sc.low:
+            out.append(x / sc.factor)
+        else:
+            s = (sc.original / wl - sc.low) / (sc.high - sc.low) if sc.high != sc.low else 1.0
+            out.append((1.0 - s) * x / sc.factor + s * x)
+    return out
+
+
+def tiny_gugezen(width=96, vocab=300, layers=None, eps=1e-5, streams=3, embed_scale=0.7, logit_scale=1.5):
+    """A small Gugezen config dict for tests: sizes deliberately unequal between layers and between the halves of a parallel mixer (dim !=
+    vdim, heads != kv_heads, partly rotated heads, state != vdim, groups != norm_groups), one layer without a feed-forward, a mixture
+    without a shared unit, two layers that use another one's tensors."""
+    rot = lambda dims, scaled, base=10000.0: {'base': base, 'dims': dims,
+                                              **({'scaling': {'factor': 4.0, 'low': 1.0, 'high': 4.0, 'original': 64}} if scaled else {})}
+    par = lambda lh, lkv, ld, lv, rd, rh, rdim, rv, ls=0.8, rs=1.1, scaled=True: {
+        'type': 'parallel',
+        'mixer': {'left': dict(heads=lh, kv_heads=lkv, dim=ld, vdim=lv, scale=2.0 * ld ** -0.5, rot=rot(rd, scaled)),
+                  'right': dict(heads=rh, dim=rdim, vdim=rv, decay=[1.0 - 2.0 ** -(1 + 1.7 * h) for h in range(rh)]),
+                  'left_scale': ls, 'right_scale': rs}}
+    mam = lambda heads, vdim, state, groups, taps, parts: {
+        'type': 'mamba2', 'mixer': dict(heads=heads, vdim=vdim, state=state, groups=groups, conv=taps, norm_groups=parts)}
+    dense = lambda ff: {'kind': 'dense', 'ff': ff}
+    moe = lambda ff, e, top, shared=None: {'kind': 'moe', 'expert': {'ff': ff}, 'router': dict(experts=e, top=top),
+                                           **({'shared': {'ff': shared}} if shared else {})}
+    if layers is None:
+        p0, m1 = dict(par(6, 3, 24, 40, 16, 3, 24, 40), mlp=moe(40, 5, 2, 72)), dict(mam(6, 24, 40, 2, 4, 3), mlp=dense(136))
+        layers = [p0, m1, dict(p0, weights_of=0), dict(mam(4, 40, 24, 4, 3, 2), mlp=None),
+                  dict(par(4, 1, 40, 24, 40, 2, 40, 72, 1.2, 0.6, False), mlp=moe(32, 4, 3)), dict(m1, weights_of=1)]
+    return {'architecture': 'Gugezen', 'vocab': vocab, 'width': width, 'norm': {'eps': eps}, 'embedding': {'scale': embed_scale},
+            'streams': streams, 'logit_scale': logit_scale, 'layers': layers}

@@ -46,6 +46,14 @@
 //   delta_scan_kernel           the layout of the linear-attention scan; two passes over the state columns per token, the sums S^T k
 //                               (a shuffle reduction closes them, on the critical path) and then update and read-out. It also moves the
 //                               convolution history on: by then no kernel of the step reads the old one.
+//
+// Memory with one decay per head and token, without the correction: S <- g_t S + b_t k_t v_t^T, y_t = S^T q_t + c v_t. This is the
+// recurrence of Mamba-2 (Dao, Gu, "Transformers are SSMs: Generalized Models and Efficient Algorithms Through Structured State Space
+// Duality": q = C, k = B, v = x, g = exp(-exp(A) dt), b = dt, heads in groups that share B and C, a skip factor c) and, with a constant
+// g per head, b = 1 and c = 0, linear attention with fixed decays.
+//   short_conv_kernel           as above, with a bias per channel; the gates are then g and b = dt
+//   delta_scan_kernel           with DELTA = false: one pass over the state columns per token
+//   part_norm_gate_kernel       rows normed in equal parts (one part: all heads together), with the gate in front of the norm or behind it
 #include "common.cuh"
 #include "../../include/phi3_b200.h"
 #include <cfloat>
@@ -426,7 +434,7 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) gla_scan_kernel(p3_gla_args a)
             if (col + c * CW < dv && d0 + j < d) Sg[(size_t)(d0 + j) * dv + col + c * CW] = S[c][j];
 }
 
-// ---------------------------------------------------------------- short convolutions, unit heads, gates of the delta rule
+// ---------------------------------------------------------------- short convolutions, unit heads, gates of the scan behind them
 template <int VEC> __device__ __forceinline__ void ldvec(const float* p, float* v) {
     if constexpr (VEC == 4) { const float4 u = *reinterpret_cast<const float4*>(p); v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w; }
     else if constexpr (VEC == 2) { const float2 u = *reinterpret_cast<const float2*>(p); v[0] = u.x; v[1] = u.y; }
@@ -449,16 +457,16 @@ __global__ void __launch_bounds__(128) short_conv_kernel(p3_short_conv_args a, i
     const int taps = TAPS > 0 ? TAPS : a.taps;
     const int C = a.n_unit * a.dim + a.n_plain;
     const int r_lo = blockIdx.x * rows_per, r_hi = min(a.n_rows, r_lo + rows_per);
-    if (job >= n_conv_jobs) {                                // gates: {decay, beta} of every head
+    if (job >= n_conv_jobs) {                                // gates: {decay, beta or step} of every head
         if (job > n_conv_jobs || !a.gates) return;
         for (int i = lane; i < (r_hi - r_lo) * a.n_gates; i += 32) {
             const int r = r_lo + i / a.n_gates, h = i % a.n_gates;
             const float* pr = a.proj + (size_t)r * a.ld_proj;
-            const float z = pr[a.a_off + h] + a.dt_bias[h], b = pr[a.b_off + h];
+            const float z = pr[a.a_off + h] + a.dt_bias[h];
             const float soft = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));              // softplus without overflow
             float* g = a.gates + ((size_t)r * a.n_gates + h) * 2;
             g[0] = expf(-expf(a.a_log[h]) * soft);
-            g[1] = 1.0f / (1.0f + expf(-b));
+            g[1] = a.gate_mode == 1 ? soft : 1.0f / (1.0f + expf(-pr[a.b_off + h]));
         }
         return;
     }
@@ -477,7 +485,10 @@ __global__ void __launch_bounds__(128) short_conv_kernel(p3_short_conv_args a, i
                 for (int e = 0; e < VEC; e++) v[k * VEC + e] = 0.f;
         }
     };
-    float w[TAPS > 0 ? TAPS : 1][N], win[WIN][N], cur[N], nxt[N];
+    float w[TAPS > 0 ? TAPS : 1][N], win[WIN][N], cur[N], nxt[N], bias[N];
+#pragma unroll
+    for (int e = 0; e < N; e++) bias[e] = 0.f;
+    if (a.bias) load(a.bias + c0, bias);
     if (TAPS > 0) {
 #pragma unroll
         for (int j = 0; j < TAPS; j++) load(a.w + (size_t)j * C + c0, w[j]);
@@ -505,7 +516,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(p3_short_conv_args a, i
         }
         float z[N];
 #pragma unroll
-        for (int e = 0; e < N; e++) z[e] = 0.f;
+        for (int e = 0; e < N; e++) z[e] = bias[e];
         if (TAPS > 0) {
 #pragma unroll
             for (int j = 0; j < TAPS - 1; j++)
@@ -545,7 +556,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(p3_short_conv_args a, i
     }
 }
 
-// ---------------------------------------------------------------- gated delta rule
+// ---------------------------------------------------------------- gated delta rule, and the same memory without the correction
 // a 16-byte shared load that the compiler does not merge with an earlier one of the same address
 __device__ __forceinline__ float4 lds_again(const float4* p) {
     float4 v;
@@ -555,7 +566,7 @@ __device__ __forceinline__ float4 lds_again(const float4* p) {
 
 __host__ __device__ inline int64_t delta_head_floats(int dim, int vdim) { return (int64_t)dim * vdim; }
 
-template <int DS, int RS, int NC, int TB>
+template <int DS, int RS, int NC, int TB, bool DELTA>
 __global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_scan_args a) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
     pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
@@ -602,7 +613,8 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_sca
             const int tt = i / COLS, c = vb * COLS + (i - tt * COLS);
             cp_async4z(smem_u32(vs + i), a.qkv + (size_t)(row0 + t0 + tt) * a.ld_qkv + a.v_off + (size_t)hd * dv + (c < dv ? c : 0), c < dv ? 4 : 0);
         }
-        for (int i = tid; i < nb * 2; i += NT) cp_async4z(smem_u32(gs + i), a.gates + ((size_t)(row0 + t0 + i / 2) * H + hd) * 2 + (i & 1), 4);
+        if (DELTA || a.gates)
+            for (int i = tid; i < nb * 2; i += NT) cp_async4z(smem_u32(gs + i), a.gates + ((size_t)(row0 + t0 + i / 2) * H + hd) * 2 + (i & 1), 4);
     };
 
     stage(0, 0);
@@ -619,6 +631,7 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_sca
                                                             : pos0 + rel >= 0 ? hist[(size_t)(j + n_tok) * a.channels + c] : 0.f;
             }
     }
+    const float fixed = DELTA || a.gates ? 0.f : a.decay[hd], skip = DELTA || !a.skip ? 0.f : a.skip[hd];
     float S[NC][DS];
 #pragma unroll
     for (int c = 0; c < NC; c++)
@@ -635,35 +648,39 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_sca
         const float* ks = qs + TB * DPP;
         const float* vs = ks + TB * DPP;
         const float* gs = vs + TB * COLS;
-#pragma unroll(DS >= 64 ? 1 : 2)
+#pragma unroll(DS >= (DELTA ? 64 : 128) ? 1 : 2)
         for (int tt = 0; tt < nb; tt++) {
-            const float keep = gs[2 * tt], beta = gs[2 * tt + 1];
+            const float keep = DELTA || a.gates ? gs[2 * tt] : fixed, beta = DELTA || a.gates ? gs[2 * tt + 1] : 1.f;
             const float4* kq = reinterpret_cast<const float4*>(ks + tt * DPP + at_row(d0));
             const float4* qq = reinterpret_cast<const float4*>(qs + tt * DPP + at_row(d0));
             float acc[NC][4], u[NC];
 #pragma unroll
             for (int c = 0; c < NC; c++) acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
+            if constexpr (DELTA) {
 #pragma unroll
-            for (int j = 0; j < DS; j += 4) {
-                const float4 kk = kq[j / 4];
+                for (int j = 0; j < DS; j += 4) {
+                    const float4 kk = kq[j / 4];
 #pragma unroll
-                for (int c = 0; c < NC; c++) {
-                    acc[c][0] = fmaf(S[c][j], kk.x, acc[c][0]);         acc[c][1] = fmaf(S[c][j + 1], kk.y, acc[c][1]);
-                    acc[c][2] = fmaf(S[c][j + 2], kk.z, acc[c][2]);     acc[c][3] = fmaf(S[c][j + 3], kk.w, acc[c][3]);
+                    for (int c = 0; c < NC; c++) {
+                        acc[c][0] = fmaf(S[c][j], kk.x, acc[c][0]);         acc[c][1] = fmaf(S[c][j + 1], kk.y, acc[c][1]);
+                        acc[c][2] = fmaf(S[c][j + 2], kk.z, acc[c][2]);     acc[c][3] = fmaf(S[c][j + 3], kk.w, acc[c][3]);
+                    }
                 }
             }
 #pragma unroll
             for (int c = 0; c < NC; c++) {
+                const float vv = vs[tt * COLS + warp * WCOLS + lane % CW + c * CW];
+                if constexpr (!DELTA) { u[c] = beta * vv; continue; }
                 float p = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
                 if (RS >= 2) p += __shfl_xor_sync(0xffffffffu, p, CW);
                 if (RS >= 4) p += __shfl_xor_sync(0xffffffffu, p, 2 * CW);
-                u[c] = beta * (vs[tt * COLS + warp * WCOLS + lane % CW + c * CW] - keep * p);   // (decay S)^T k = decay (S^T k)
+                u[c] = beta * (vv - keep * p);             // (decay S)^T k = decay (S^T k)
                 acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
             }
 #pragma unroll
             for (int j = 0; j < DS; j += 4) {
                 // up to 32 rows per lane the k row stays in registers between the passes
-                const float4 kk = DS <= 32 ? kq[j / 4] : lds_again(kq + j / 4), qv = qq[j / 4];
+                const float4 kk = DS <= 32 || !DELTA ? kq[j / 4] : lds_again(kq + j / 4), qv = qq[j / 4];
 #pragma unroll
                 for (int c = 0; c < NC; c++) {
                     S[c][j] = fmaf(kk.x, u[c], keep * S[c][j]);         acc[c][0] = fmaf(S[c][j], qv.x, acc[c][0]);
@@ -677,6 +694,7 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_sca
                 float y = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
                 if (RS >= 2) y += __shfl_xor_sync(0xffffffffu, y, CW);
                 if (RS >= 4) y += __shfl_xor_sync(0xffffffffu, y, 2 * CW);
+                if (!DELTA) y = fmaf(skip, vs[tt * COLS + warp * WCOLS + lane % CW + c * CW], y);
                 if (lane < CW && col + c * CW < dv)
                     a.out[(size_t)(row0 + t0 + tt) * a.ld_out + (size_t)hd * dv + col + c * CW] = y;
             }
@@ -726,6 +744,68 @@ __global__ void headnorm_gate_kernel(const float* __restrict__ y, int64_t ldy, c
         const int c = h * dv + i;
         stv(out + t * ldo + c, yr[i] / dn * r * gain[gain_shared ? i : c] * gated(c));
     }
+}
+
+// One job = one part (n numbers) of a row: a warp (WARP, four jobs per CTA) or a whole CTA. Up to PN numbers per thread stay in registers,
+// VEC neighbours loaded and stored together.
+constexpr int PN = 8;
+template <typename AT, int VEC, bool WARP>
+__global__ void part_norm_gate_kernel(const float* __restrict__ y, int64_t ldy, int parts, int n, const float* __restrict__ gain,
+                                      const float* __restrict__ gate, int64_t ld_gate, int gate_silu, int gate_first, float scale, float eps,
+                                      AT* __restrict__ out, int64_t ldo, int64_t T) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    __shared__ float sh[32];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int nt = WARP ? 32 : blockDim.x, me = WARP ? lane : threadIdx.x;
+    const int64_t job = WARP ? blockIdx.x * (int64_t)(blockDim.x >> 5) + warp : blockIdx.x;
+    if (WARP && job >= T * parts) return;
+    const int64_t t = job / parts;
+    const int c0 = (int)(job - t * parts) * n;
+    const float* yr = y + t * ldy + c0;
+    const float* gr = gate ? gate + t * ld_gate + c0 : nullptr;
+    const float* wr = gain + c0;
+    AT* o = out + t * ldo + c0;
+    auto at = [&](int k) { return ((k / VEC) * nt + me) * VEC + k % VEC; };
+    auto act = [&](float g) { const float s = 1.0f / (1.0f + expf(-g)); return gate_silu ? g * s : s; };
+    float v[PN], g[PN];
+#pragma unroll
+    for (int k = 0; k < PN; k += VEC) {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) { v[k + e] = 0.f; g[k + e] = 0.f; }
+        const int i = at(k);
+        if (i < n) { ldvec<VEC>(yr + i, v + k); if (gr) ldvec<VEC>(gr + i, g + k); }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PN; k++) {
+        g[k] = gr ? act(g[k]) : 1.f;
+        if (gate_first) v[k] *= g[k];
+        ss = fmaf(v[k], v[k], ss);
+    }
+    auto first = [&](int i) { return gate_first && gr ? yr[i] * act(gr[i]) : yr[i]; };
+    for (int i = me + PN * nt; i < n; i += nt) { const float u = first(i); ss = fmaf(u, u, ss); }
+    ss = warp_sum(ss);
+    if (!WARP) {
+        if (lane == 0) sh[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
+        for (int w = 0; w < (int)(blockDim.x >> 5); w++) ss += sh[w];
+    }
+    const float r = scale / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int k = 0; k < PN; k += VEC) {
+        const int i = at(k);
+        if (i >= n) continue;
+        float w[VEC];
+        ldvec<VEC>(wr + i, w);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) w[e] = v[k + e] * r * w[e] * (gate_first ? 1.f : g[k + e]);
+        if constexpr (VEC == 4 && sizeof(AT) == 2) *reinterpret_cast<uint2*>(o + i) = make_uint2(pack_bf16(w[0], w[1]), pack_bf16(w[2], w[3]));
+        else if constexpr (VEC == 4) stvec<4>((float*)o + i, w);
+        else stv(o + i, w[0]);
+    }
+    for (int i = me + PN * nt; i < n; i += nt) stv(o + i, first(i) * r * wr[i] * (gr && !gate_first ? act(gr[i]) : 1.f));
 }
 template <typename K>
 int set_smem_attr(K kernel, size_t bytes) {
@@ -788,6 +868,28 @@ extern "C" int p3_headnorm_gate(const float* y, int64_t ldy, const float* den, i
     return p3_headnorm_gate_x(y, ldy, den, n_heads, vdim, gain, 0, gate, ld_gate, 0, scale, eps, out, ldo, out_f32, T, st);
 }
 
+extern "C" int p3_part_norm_gate(const float* y, int64_t ldy, int parts, int n, const float* gain, const float* gate, int64_t ld_gate,
+                                 int gate_silu, int gate_first, float scale, float eps, void* out, int64_t ldo, int out_f32, int64_t T,
+                                 cudaStream_t st) {
+    P3_CHECK_ARG(y && gain && out && parts >= 1 && n >= 1, "part_norm_gate: null argument");
+    if (T == 0) return 0;
+    const bool vec = n % 4 == 0 && ldy % 4 == 0 && (!gate || ld_gate % 4 == 0) && ldo % 4 == 0 &&
+                     (((uintptr_t)y | (uintptr_t)gain | (uintptr_t)gate) & 15) == 0 && ((uintptr_t)out & (out_f32 ? 15 : 7)) == 0;
+    const int64_t jobs = T * parts;
+    const bool warp = n <= 32 * PN;
+    int th = (n + PN * 32 - 1) / (PN * 32) * 32;             // threads whose registers hold a part of n numbers (up to 8192)
+    th = warp ? 128 : th > 1024 ? 1024 : th;
+    const unsigned grid = (unsigned)(warp ? (jobs + 3) / 4 : jobs);
+#define GO(AT, V, WP) p3_launch_pdl(part_norm_gate_kernel<AT, V, WP>, dim3(grid), dim3(th), (size_t)(0), st, y, ldy, parts, n, gain, gate, ld_gate, \
+                                    gate_silu, gate_first, scale, eps, (AT*)out, ldo, T)
+#define GV(AT) do { if (vec) { if (warp) GO(AT, 4, true); else GO(AT, 4, false); } else { if (warp) GO(AT, 1, true); else GO(AT, 1, false); } } while (0)
+    if (out_f32) GV(float); else GV(bf16);
+#undef GV
+#undef GO
+    P3_CHECK_LAUNCH("part_norm_gate");
+    return 0;
+}
+
 extern "C" int64_t p3_gla_state_floats(int n_heads, int dim, int vdim) { return (int64_t)n_heads * gla_head_floats(dim, vdim); }
 
 extern "C" int p3_gla_scan(const p3_gla_args* a, cudaStream_t st) {
@@ -847,13 +949,14 @@ extern "C" int p3_short_conv(const p3_short_conv_args* a, cudaStream_t st) {
     P3_CHECK_ARG(a->n_unit >= 0 && a->n_plain >= 0 && a->n_scaled <= a->n_unit && (a->n_unit == 0 || (a->dim >= 1 && a->dim <= 512)),
                  "short_conv: need 1 <= dim <= 512 and n_scaled <= n_unit");
     P3_CHECK_ARG(!a->gates || (a->n_gates >= 1 && a->a_log && a->dt_bias), "short_conv: the gates need a_log and dt_bias");
+    P3_CHECK_ARG(a->gate_mode == 0 || a->gate_mode == 1, "short_conv: gate_mode is 0 (decay, beta) or 1 (decay, step)");
     P3_CHECK_ARG(((uintptr_t)a->seqs & 15) == 0, "short_conv: the sequence records must be 16-byte aligned");
     if (a->n_rows == 0) return 0;
     const int d = a->n_unit ? a->dim : 128, C = a->n_unit * a->dim + a->n_plain;
     auto fits = [&](int v) {                                 // may a lane take v neighbouring channels at once?
         const uintptr_t m = (uintptr_t)v * 4 - 1;
         return d % v == 0 && C % v == 0 && a->c_off % v == 0 && a->ld_proj % v == 0 && a->ld_out % v == 0 &&
-               (((uintptr_t)a->proj | (uintptr_t)a->w | (uintptr_t)a->out | (uintptr_t)a->conv_state) & m) == 0;
+               (((uintptr_t)a->proj | (uintptr_t)a->w | (uintptr_t)a->bias | (uintptr_t)a->out | (uintptr_t)a->conv_state) & m) == 0;
     };
     const int vec = d > 64 && fits(4) ? 4 : d > 32 && fits(2) ? 2 : 1;
     const int need = (d + 32 * vec - 1) / (32 * vec), nv = need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : need <= 8 ? 8 : 16;
@@ -873,12 +976,14 @@ extern "C" int p3_short_conv(const p3_short_conv_args* a, cudaStream_t st) {
 
 extern "C" int64_t p3_delta_state_floats(int n_heads, int dim, int vdim) { return (int64_t)n_heads * delta_head_floats(dim, vdim); }
 
-extern "C" int p3_delta_scan(const p3_delta_scan_args* a, cudaStream_t st) {
-    P3_CHECK_ARG(a && a->qkv && a->gates && a->state && a->seqs && a->out, "delta_scan: null argument");
-    P3_CHECK_ARG(a->n_heads >= 1 && a->n_kv >= 1 && a->n_heads % a->n_kv == 0, "delta_scan: heads must be a multiple of kv heads");
-    P3_CHECK_ARG(a->dim >= 1 && a->dim <= 512 && a->vdim >= 1, "delta_scan: need 1 <= dim <= 512, vdim >= 1");
-    P3_CHECK_ARG(a->taps <= 1 || (a->conv_in && a->conv_state && a->channels >= 1), "delta_scan: the convolution history needs its inputs");
-    P3_CHECK_ARG(((uintptr_t)a->seqs & 15) == 0, "delta_scan: the sequence records must be 16-byte aligned");
+namespace {
+template <bool DELTA>
+int launch_scan(const p3_delta_scan_args* a, cudaStream_t st, const char* who) {
+    P3_CHECK_ARG(a && a->qkv && a->state && a->seqs && a->out, "%s: null argument", who);
+    P3_CHECK_ARG(a->n_heads >= 1 && a->n_kv >= 1 && a->n_heads % a->n_kv == 0, "%s: heads must be a multiple of kv heads", who);
+    P3_CHECK_ARG(a->dim >= 1 && a->dim <= 512 && a->vdim >= 1, "%s: need 1 <= dim <= 512, vdim >= 1", who);
+    P3_CHECK_ARG(a->taps <= 1 || (a->conv_in && a->conv_state && a->channels >= 1), "%s: the convolution history needs its inputs", who);
+    P3_CHECK_ARG(((uintptr_t)a->seqs & 15) == 0, "%s: the sequence records must be 16-byte aligned", who);
     if (a->n_seqs == 0) return 0;
     // A warp is four row slices x eight lanes, a lane owns one or two columns: the choice of the linear-attention scan
     int rs = 4, nc = (int64_t)a->n_seqs * a->n_heads * ((a->vdim + 31) / 32) > 148 ? 2 : 1;
@@ -890,13 +995,24 @@ extern "C" int p3_delta_scan(const p3_delta_scan_args* a, cudaStream_t st) {
     const dim3 grid((unsigned)a->n_seqs, (unsigned)a->n_heads, (unsigned)((a->vdim + cols - 1) / cols));
     const size_t bytes = sizeof(float) * (size_t)2 * tb * (2 * (ds * rs + 4 * rs) + cols + 2);   // two staged rounds
 #define GO(DS, RS, NC, TB)                                                                                             \
-    do { if (set_smem_attr(delta_scan_kernel<DS, RS, NC, TB>, bytes)) return -1;                                         \
-         p3_launch_pdl(delta_scan_kernel<DS, RS, NC, TB>, dim3(grid), dim3(GLA_WARPS * 32), (size_t)(bytes), st, *a); } while (0)
+    do { if (set_smem_attr(delta_scan_kernel<DS, RS, NC, TB, DELTA>, bytes)) return -1;                                  \
+         p3_launch_pdl(delta_scan_kernel<DS, RS, NC, TB, DELTA>, dim3(grid), dim3(GLA_WARPS * 32), (size_t)(bytes), st, *a); } while (0)
     if (a->dim > 256) GO(128, 4, 1, 16);
     else if (rs == 2) { if (ds == 16) GO(16, 2, 1, MM_TB); else if (ds == 32) GO(32, 2, 1, MM_TB); else if (ds == 64) GO(64, 2, 1, MM_TB); else GO(128, 2, 1, MM_TB); }
     else if (nc == 1) { if (ds == 16) GO(16, 4, 1, MM_TB); else if (ds == 32) GO(32, 4, 1, MM_TB); else GO(64, 4, 1, MM_TB); }
     else { if (ds == 16) GO(16, 4, 2, MM_TB); else if (ds == 32) GO(32, 4, 2, MM_TB); else GO(64, 4, 2, MM_TB); }
 #undef GO
-    P3_CHECK_LAUNCH("delta_scan");
+    P3_CHECK_LAUNCH(who);
     return 0;
+}
+}  // namespace
+
+extern "C" int p3_delta_scan(const p3_delta_scan_args* a, cudaStream_t st) {
+    P3_CHECK_ARG(a && a->gates, "delta_scan: null argument");
+    return launch_scan<true>(a, st, "delta_scan");
+}
+
+extern "C" int p3_decay_scan(const p3_delta_scan_args* a, cudaStream_t st) {
+    P3_CHECK_ARG(a && (a->gates || a->decay), "decay_scan: needs gates, or one decay per head");
+    return launch_scan<false>(a, st, "decay_scan");
 }

@@ -4,8 +4,8 @@
 // gated-linear activation, the mixture-of-experts router (logits, top-k, softmax over the chosen), the expert sort and the
 // weighted combine, the distance tables of the biased attention (logarithmic and linear), and the embedding that adds the row of
 // a hashed (previous, current) token pair, with the previous token kept per sequence slot; the embedding under a norm and the
-// residual add with one norm behind it. Everything here is fp32 arithmetic; only the
-// storage type of activations ("act": bf16 or fp32) and of the cache differs between the serving mode and the all-fp32 mode.
+// residual add with one norm behind it; several residual streams per token that are mixed around every sublayer. Everything here is
+// fp32 arithmetic; only the storage type of activations ("act": bf16 or fp32) and of the cache differs between the serving mode and the all-fp32 mode.
 #include "common.cuh"
 #include "../../include/phi3_b200.h"
 
@@ -522,8 +522,13 @@ __global__ void latent_post_kernel(p3_latent_post_args a) {
     }
 }
 
-// ---------------------------------------------------------------- y = act(g) * u, act = silu or relu
-template <int ACT> __device__ __forceinline__ float glu_act(float g) { return ACT == 0 ? g / (1.0f + expf(-g)) : fmaxf(g, 0.f); }
+// ---------------------------------------------------------------- y = act(g) * u, act = silu, relu or the tanh form of gelu
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+template <int ACT> __device__ __forceinline__ float glu_act(float g) {
+    return ACT == 0 ? g / (1.0f + expf(-g)) : ACT == 1 ? fmaxf(g, 0.f) : gelu_tanh(g);
+}
+template <int ACT> __device__ __forceinline__ float unit_act(float z) { return ACT == 0 ? gelu_erf(z) : gelu_tanh(z); }
 
 template <typename AT, int ACT>
 __global__ void glu_kernel(const float* __restrict__ g, const float* __restrict__ u, int64_t ld, AT* __restrict__ out, int64_t ldo,
@@ -550,6 +555,35 @@ __global__ void glu_vec4_kernel(const float* __restrict__ g, const float* __rest
         const float4 gv = *reinterpret_cast<const float4*>(g + (size_t)r * ld + c), uv = *reinterpret_cast<const float4*>(u + (size_t)r * ld + c);
         const float y0 = glu_act<ACT>(gv.x) * uv.x, y1 = glu_act<ACT>(gv.y) * uv.y;
         const float y2 = glu_act<ACT>(gv.z) * uv.z, y3 = glu_act<ACT>(gv.w) * uv.w;
+        AT* o = out + (size_t)r * ldo + c;
+        if constexpr (sizeof(AT) == 4) *reinterpret_cast<float4*>(o) = make_float4(y0, y1, y2, y3);
+        else *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(y0, y1), pack_bf16(y2, y3));
+    }
+}
+
+// ---------------------------------------------------------------- y = act(u), a unit without a gate; act = gelu (erf) or its tanh form
+template <typename AT, int ACT>
+__global__ void unit_act_kernel(const float* __restrict__ u, int64_t ld, AT* __restrict__ out, int64_t ldo, int64_t R, int F) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    const int64_t n = R * F;
+    for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t r = i / F; const int c = (int)(i % F);
+        stv(out + (size_t)r * ldo + c, unit_act<ACT>(u[(size_t)r * ld + c]));
+    }
+}
+
+// four columns per thread (F, the row pitches and the pointers are multiples of four elements): 16-byte loads
+template <typename AT, int ACT>
+__global__ void unit_act_vec4_kernel(const float* __restrict__ u, int64_t ld, AT* __restrict__ out, int64_t ldo, int64_t R, int F) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    const int F4 = F / 4;
+    const int64_t n = R * F4;
+    for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t r = i / F4; const int c = (int)(i % F4) * 4;
+        const float4 v = *reinterpret_cast<const float4*>(u + (size_t)r * ld + c);
+        const float y0 = unit_act<ACT>(v.x), y1 = unit_act<ACT>(v.y), y2 = unit_act<ACT>(v.z), y3 = unit_act<ACT>(v.w);
         AT* o = out + (size_t)r * ldo + c;
         if constexpr (sizeof(AT) == 4) *reinterpret_cast<float4*>(o) = make_float4(y0, y1, y2, y3);
         else *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(y0, y1), pack_bf16(y2, y3));
@@ -753,9 +787,10 @@ __global__ void token_shift_kernel(const float* __restrict__ h, const float* __r
 // ---------------------------------------------------------------- rotation of q and k + paged K/V write (+ projection biases, unit norm)
 // Grid (token, job group): one warp per head job (H query heads, G key heads, G value heads when there is a value projection).
 // The CTA forms cos and sin of its token's angles once, in shared memory: position * frequency in fp32 with the full-range
-// sincosf. The lane that owns number i < rot_n / 2 of a head also owns its partner i + rot_n / 2. Without a value projection the
-// key head is written twice: rotated to the K pool, as projected to the V pool. The root mean square of the unit norm is taken
-// from the numbers before they turn: a rotation keeps the length of a pair, so its squares count with the factor mag^2.
+// sincosf. A turning pair is numbers i and i + rot_n / 2, or neighbours 2i and 2i + 1 (pair_mode 1); one lane owns both. Without a
+// value projection the key head is written twice: rotated to the K pool, as projected to the V pool. The root mean square of the
+// unit norm is taken from the numbers before they turn: a rotation keeps the length of a pair, so its squares count with the factor
+// mag^2. The columns of a recurrent mixer that shares the projection can pass silu on the way, in place.
 template <typename AT, typename CT>
 __global__ void qkv_rope_kv_write_kernel(p3_qkv_rope_post_args a) {
     pdl_trigger();                                           // the next kernel may set up while this one runs ...
@@ -773,6 +808,20 @@ __global__ void qkv_rope_kv_write_kernel(p3_qkv_rope_post_args a) {
         turn[i] = make_float2(cs * mag, sn * mag);
     }
     __syncthreads();
+    if (a.n_act > 0) {                                       // silu in place; the row's CTAs share the columns
+        float* ac = a.act_cols + (size_t)t * a.ld_proj;
+        const int me = blockIdx.y * blockDim.x + threadIdx.x, n_thr = gridDim.y * blockDim.x;
+        if (a.n_act % 4 == 0 && a.ld_proj % 4 == 0 && ((uintptr_t)a.act_cols & 15) == 0) {
+            for (int i = me * 4; i < a.n_act; i += n_thr * 4) {
+                float4 v = *reinterpret_cast<float4*>(ac + i);
+                v.x = v.x / (1.0f + expf(-v.x)); v.y = v.y / (1.0f + expf(-v.y));
+                v.z = v.z / (1.0f + expf(-v.z)); v.w = v.w / (1.0f + expf(-v.w));
+                *reinterpret_cast<float4*>(ac + i) = v;
+            }
+        } else {
+            for (int i = me; i < a.n_act; i += n_thr) ac[i] = ac[i] / (1.0f + expf(-ac[i]));
+        }
+    }
     const bool v_is_k = a.v_off < 0;
     const int jobs = H + G + (v_is_k ? 0 : G);
     for (int job = blockIdx.y * nw + warp; job < jobs; job += gridDim.y * nw) {
@@ -793,6 +842,20 @@ __global__ void qkv_rope_kv_write_kernel(p3_qkv_rope_post_args a) {
                     if (i < a.rot_n) st = fmaf(u, u, st); else sp = fmaf(u, u, sp);
                 }
                 r = 1.0f / sqrtf(warp_sum(fmaf(st, mag * mag, sp)) / (float)d + a.eps);
+            }
+            if (a.pair_mode) {                               // neighbours turn together: a lane walks pairs (2i, 2i + 1)
+                for (int i = 2 * lane; i < d; i += 64) {
+                    const bool two = i + 1 < d;
+                    const float u = src[i] + (b ? b[i] : 0.f), w = two ? src[i + 1] + (b ? b[i + 1] : 0.f) : 0.f;
+                    const float2 cs = i < a.rot_n ? turn[i / 2] : make_float2(1.f, 0.f);
+                    const float r0 = (u * cs.x - w * cs.y) * r, r1 = (w * cs.x + u * cs.y) * r;
+                    if (isq) { stv(dq + i, r0); if (two) stv(dq + i + 1, r1); }
+                    else {
+                        stv(dk + i, r0); if (two) stv(dk + i + 1, r1);
+                        if (dvv) { stv(dvv + i, u); if (two) stv(dvv + i + 1, w); }
+                    }
+                }
+                continue;
             }
             for (int i = lane; i < d; i += 32) {
                 if (i >= half && i < a.rot_n) continue;      // the partner of a turning pair: written by the pair's owner
@@ -1083,6 +1146,168 @@ __global__ void residual_rmsnorm_kernel(float* x, const float* __restrict__ y, i
     }
 }
 
+// ---------------------------------------------------------------- several residual streams per token (hyper-connections)
+// x [T][S][W]. One CTA per row. With a sublayer output y every column takes X_t <- sum_s M[s][t] X_s + b_t y, all streams from the old
+// ones; then u = sum_s a_s X_s of the new streams, whose root mean square is the only thing the columns share. Up to RPT numbers of u
+// per thread stay in registers between the statistic and the write; the old streams of a few columns are held at a time. More than four streams: column by column through memory.
+template <typename AT, int SMAX, int VEC>
+__global__ void __launch_bounds__(1024) streams_rmsnorm_kernel(float* x, int S, const float* __restrict__ y, int64_t ldy,
+                                                               const float* __restrict__ mix, const float* __restrict__ out_w,
+                                                               const float* __restrict__ in_w, const int32_t* __restrict__ rows,
+                                                               const float* __restrict__ gain, AT* __restrict__ h, int W, float eps) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    constexpr int CH = SMAX <= 2 ? RPT : VEC;                // numbers per thread whose old streams are loaded at once
+    constexpr int RP = SMAX <= 4 ? RPT : 0;                  // numbers of u per thread in registers
+    __shared__ float sh[32], M[SMAX * SMAX], B[SMAX], A[SMAX];   // M [from][to]; zeros beyond S
+    const int64_t r = blockIdx.x, t = rows ? rows[r] : r;
+    float* xr = x + (size_t)t * S * W;
+    const float* yr = y ? y + (size_t)t * ldy : nullptr;
+    const int nt = blockDim.x;
+    for (int i = threadIdx.x; i < SMAX * SMAX; i += nt) M[i] = (yr && i / SMAX < S && i % SMAX < S) ? mix[i / SMAX * S + i % SMAX] : 0.f;
+    for (int i = threadIdx.x; i < SMAX; i += nt) { A[i] = (gain && i < S) ? in_w[i] : 0.f; B[i] = (yr && i < S) ? out_w[i] : 0.f; }
+    __syncthreads();
+    float v[RPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int k0 = 0; k0 < RP; k0 += CH) {
+        float o[SMAX][CH], yv[CH];
+#pragma unroll
+        for (int k = 0; k < CH; k += VEC) {
+            const int i = row_at<VEC>(k0 + k);
+#pragma unroll
+            for (int s = 0; s < SMAX; s++) {
+                if constexpr (VEC == 4) {
+                    const float4 u = (i < W && s < S) ? *reinterpret_cast<const float4*>(xr + (size_t)s * W + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    o[s][k] = u.x; o[s][k + 1] = u.y; o[s][k + 2] = u.z; o[s][k + 3] = u.w;
+                } else o[s][k] = (i < W && s < S) ? xr[(size_t)s * W + i] : 0.f;
+            }
+            if (yr) {
+                if constexpr (VEC == 4) {
+                    const float4 u = i < W ? *reinterpret_cast<const float4*>(yr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    yv[k] = u.x; yv[k + 1] = u.y; yv[k + 2] = u.z; yv[k + 3] = u.w;
+                } else yv[k] = i < W ? yr[i] : 0.f;
+            }
+        }
+        if (yr) {
+#pragma unroll
+            for (int k = 0; k < CH; k++) v[k0 + k] = 0.f;
+#pragma unroll
+            for (int to = 0; to < SMAX; to++) {
+                float n[CH];
+#pragma unroll
+                for (int k = 0; k < CH; k++) {
+                    n[k] = B[to] * yv[k];
+#pragma unroll
+                    for (int s = 0; s < SMAX; s++) n[k] = fmaf(M[s * SMAX + to], o[s][k], n[k]);
+                    v[k0 + k] = fmaf(A[to], n[k], v[k0 + k]);
+                }
+                if (!rows && to < S) {
+#pragma unroll
+                    for (int k = 0; k < CH; k += VEC) {
+                        const int i = row_at<VEC>(k0 + k);
+                        if (i < W) {
+                            if constexpr (VEC == 4) *reinterpret_cast<float4*>(xr + (size_t)to * W + i) = make_float4(n[k], n[k + 1], n[k + 2], n[k + 3]);
+                            else xr[(size_t)to * W + i] = n[k];
+                        }
+                    }
+                }
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < CH; k++) {
+                v[k0 + k] = 0.f;
+#pragma unroll
+                for (int s = 0; s < SMAX; s++) v[k0 + k] = fmaf(A[s], o[s][k], v[k0 + k]);
+            }
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < RP; k++) ss = fmaf(v[k], v[k], ss);
+    // columns beyond the registers: formed one by one, and (unless they are stored) once more when they are normed
+    auto column = [&](int i, bool store) {
+        float o[SMAX], u = 0.f;
+#pragma unroll
+        for (int s = 0; s < SMAX; s++) o[s] = s < S ? xr[(size_t)s * W + i] : 0.f;
+        const float yi = yr ? yr[i] : 0.f;
+#pragma unroll
+        for (int to = 0; to < SMAX; to++) {
+            float n = o[to];
+            if (yr) {
+                n = B[to] * yi;
+#pragma unroll
+                for (int s = 0; s < SMAX; s++) n = fmaf(M[s * SMAX + to], o[s], n);
+                if (store && to < S) xr[(size_t)to * W + i] = n;
+            }
+            u = fmaf(A[to], n, u);
+        }
+        return u;
+    };
+    const bool store = !rows && yr;
+    for (int i = threadIdx.x + RP * nt; i < W; i += nt) { const float u = column(i, store); ss = fmaf(u, u, ss); }
+    if (!gain) return;
+    ss = block_sum(ss, sh);
+    const float sc = 1.0f / sqrtf(ss / (float)W + eps);
+    if constexpr (RP > 0) {
+        float gv[RPT];
+        row_load<VEC>(gain, W, gv);
+#pragma unroll
+        for (int k = 0; k < RPT; k++) v[k] = v[k] * sc * gv[k];
+        row_store<VEC>(h + (size_t)r * W, W, v);
+    }
+    for (int i = threadIdx.x + RP * nt; i < W; i += nt) {
+        float u = 0.f;
+        if (store) { for (int s = 0; s < S; s++) u = fmaf(A[s], xr[(size_t)s * W + i], u); }   // this thread's own writes
+        else u = column(i, false);
+        stv(h + (size_t)r * W + i, u * sc * gain[i]);
+    }
+}
+
+// the start of the streams: X_s = table[id] * scale for every s, and the first sublayer's input, the norm of (sum_s a_s) X_1
+template <typename AT, int VEC>
+__global__ void embed_streams_kernel(const bf16* __restrict__ table, const int32_t* __restrict__ ids, float scale, float* __restrict__ x, int S,
+                                     const float* __restrict__ in_w, const float* __restrict__ gain, AT* __restrict__ h, int W, int vocab, float eps) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    __shared__ float sh[32];
+    const int64_t t = blockIdx.x;
+    int id = ids[t];
+    if (id < 0 || id >= vocab) id = 0;
+    const bf16* src = table + (size_t)id * W;
+    float* xr = x + (size_t)t * S * W;
+    const int nt = blockDim.x;
+    float as = 0.f;
+    for (int s = 0; s < S; s++) as += in_w[s];
+    float v[RPT], gv[RPT];
+    row_load<VEC>(gain, W, gv);
+#pragma unroll
+    for (int k = 0; k < RPT; k += VEC) {
+        const int i = row_at<VEC>(k);
+        if constexpr (VEC == 4) {
+            const uint2 u = i < W ? *reinterpret_cast<const uint2*>(src + i) : make_uint2(0u, 0u);
+            const float2 lo = unpack_bf16(u.x), hi = unpack_bf16(u.y);
+            v[k] = lo.x; v[k + 1] = lo.y; v[k + 2] = hi.x; v[k + 3] = hi.y;
+        } else v[k] = i < W ? __bfloat162float(src[i]) : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < RPT; k++) v[k] *= scale;
+    for (int s = 0; s < S; s++) row_store<VEC>(xr + (size_t)s * W, W, v);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < RPT; k++) { v[k] *= as; ss = fmaf(v[k], v[k], ss); }
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) {
+        const float e = __bfloat162float(src[i]) * scale, u = e * as;
+        for (int s = 0; s < S; s++) xr[(size_t)s * W + i] = e;
+        ss = fmaf(u, u, ss);
+    }
+    ss = block_sum(ss, sh);
+    const float sc = 1.0f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < RPT; k++) v[k] = v[k] * sc * gv[k];
+    row_store<VEC>(h + (size_t)t * W, W, v);
+    for (int i = threadIdx.x + RPT * nt; i < W; i += nt) stv(h + (size_t)t * W + i, __bfloat162float(src[i]) * scale * as * sc * gain[i]);
+}
+
 __global__ void distance_linear_kernel(const float* __restrict__ slope, float* __restrict__ pen, int H, int n) {
     const int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x;
     if (i >= (int64_t)H * n) return;
@@ -1237,14 +1462,15 @@ extern "C" int p3_latent_post(const p3_latent_post_args* a, cudaStream_t st) {
 
 extern "C" int p3_glu_act(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, int act,
                           cudaStream_t st) {
-    P3_CHECK_ARG(act == 0 || act == 1, "glu_act: the activation is 0 (silu) or 1 (relu)");
+    P3_CHECK_ARG(act >= 0 && act <= 2, "glu_act: the activation is 0 (silu), 1 (relu) or 2 (gelu, tanh form)");
     if (R == 0 || F == 0) return 0;
     const bool vec = F % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)g & 15) == 0 && ((uintptr_t)u & 15) == 0 &&
                      ((uintptr_t)out & 15) == 0;
     const int64_t n = vec ? R * (F / 4) : R * F;
     const unsigned grid = (unsigned)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
 #define GO(K, AT) do { if (act == 0) p3_launch_pdl(K<AT, 0>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (AT*)out, ldo, R, F);   \
-                       else p3_launch_pdl(K<AT, 1>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (AT*)out, ldo, R, F); } while (0)
+                       else if (act == 1) p3_launch_pdl(K<AT, 1>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (AT*)out, ldo, R, F); \
+                       else p3_launch_pdl(K<AT, 2>, dim3(grid), dim3(256), (size_t)(0), st, g, u, ld, (AT*)out, ldo, R, F); } while (0)
     if (vec) { if (out_f32) GO(glu_vec4_kernel, float); else GO(glu_vec4_kernel, bf16); }
     else { if (out_f32) GO(glu_kernel, float); else GO(glu_kernel, bf16); }
 #undef GO
@@ -1255,6 +1481,21 @@ extern "C" int p3_glu_act(const float* g, const float* u, int64_t ld, void* out,
 extern "C" int p3_glu_silu(const float* g, const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F,
                            cudaStream_t st) {
     return p3_glu_act(g, u, ld, out, ldo, out_f32, R, F, 0, st);
+}
+
+extern "C" int p3_unit_act(const float* u, int64_t ld, void* out, int64_t ldo, int out_f32, int64_t R, int F, int act, cudaStream_t st) {
+    P3_CHECK_ARG(act == 0 || act == 1, "unit_act: the activation is 0 (gelu) or 1 (gelu, tanh form)");
+    if (R == 0 || F == 0) return 0;
+    const bool vec = F % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)u | (uintptr_t)out) & 15) == 0;
+    const int64_t n = vec ? R * (F / 4) : R * F;
+    const unsigned grid = (unsigned)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+#define GO(K, AT) do { if (act == 0) p3_launch_pdl(K<AT, 0>, dim3(grid), dim3(256), (size_t)(0), st, u, ld, (AT*)out, ldo, R, F);   \
+                       else p3_launch_pdl(K<AT, 1>, dim3(grid), dim3(256), (size_t)(0), st, u, ld, (AT*)out, ldo, R, F); } while (0)
+    if (vec) { if (out_f32) GO(unit_act_vec4_kernel, float); else GO(unit_act_vec4_kernel, bf16); }
+    else { if (out_f32) GO(unit_act_kernel, float); else GO(unit_act_kernel, bf16); }
+#undef GO
+    P3_CHECK_LAUNCH("unit_act");
+    return 0;
 }
 
 extern "C" int p3_router_sigmoid_groups(const void* x, int64_t ldx, int x_f32, const float* Wr, const float* correction,
@@ -1332,6 +1573,7 @@ extern "C" int p3_qkv_rope_post(const p3_qkv_rope_post_args* a, cudaStream_t st)
     P3_CHECK_ARG(a->rot_n >= 0 && a->rot_n % 2 == 0 && a->rot_n <= a->dim && (a->rot_n == 0 || a->freq), "qkv_rope_post: rot_n must be even and <= dim, with frequencies");
     P3_CHECK_ARG(a->v_off >= 0 || a->vdim == a->dim, "qkv_rope_post: keys that double as values need vdim == dim");
     P3_CHECK_ARG(a->rot_n <= 8192, "qkv_rope_post: at most 8192 turning numbers per head");
+    P3_CHECK_ARG(a->n_act >= 0 && (a->n_act == 0 || a->act_cols), "qkv_rope_post: the silu columns need their address");
     if (a->T == 0) return 0;
     const int jobs = a->n_heads + a->n_kv + (a->v_off < 0 ? 0 : a->n_kv), th = 128;
     const int groups = a->T >= 1024 ? 1 : (jobs + 3) / 4;
@@ -1430,5 +1672,37 @@ extern "C" int p3_residual_rmsnorm(float* x, const float* y, int64_t ldy, float 
     else { if (vec) GO(bf16, 4); else GO(bf16, 1); }
 #undef GO
     P3_CHECK_LAUNCH("residual_rmsnorm");
+    return 0;
+}
+
+extern "C" int p3_embed_streams(const void* table, const int32_t* ids, float scale, float* x, int S, const float* in_w, const float* gain,
+                                void* h, int act_f32, int64_t T, int W, int vocab, float eps, cudaStream_t st) {
+    P3_CHECK_ARG(table && ids && x && in_w && gain && h && S >= 1, "embed_streams: null argument");
+    if (T == 0) return 0;
+    const int th = row_threads(W);
+    const bool vec = W % 4 == 0 && (((uintptr_t)x | (uintptr_t)gain | (uintptr_t)h) & 15) == 0 && ((uintptr_t)table & 7) == 0;
+#define GO(AT, V) p3_launch_pdl(embed_streams_kernel<AT, V>, dim3((unsigned)T), dim3(th), (size_t)(0), st, (const bf16*)table, ids, scale, x, S, in_w, gain, (AT*)h, W, vocab, eps)
+    if (act_f32) { if (vec) GO(float, 4); else GO(float, 1); }
+    else { if (vec) GO(bf16, 4); else GO(bf16, 1); }
+#undef GO
+    P3_CHECK_LAUNCH("embed_streams");
+    return 0;
+}
+
+extern "C" int p3_streams_rmsnorm(float* x, int S, const float* y, int64_t ldy, const float* mix, const float* out_w, const float* in_w,
+                                  const int32_t* rows, const float* gain, void* h, int act_f32, int64_t R, int W, float eps, cudaStream_t st) {
+    P3_CHECK_ARG(x && W >= 1 && (!y || (mix && out_w)) && (!gain || (in_w && h)), "streams_rmsnorm: null argument");
+    P3_CHECK_ARG(S >= 1 && S <= 16, "streams_rmsnorm: 1 to 16 streams");
+    if (R == 0) return 0;
+    const int th = row_threads(W);
+    const bool vec = W % 4 == 0 && (!y || ldy % 4 == 0) && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)gain | (uintptr_t)h) & 15) == 0;
+#define GO(AT, N, V) p3_launch_pdl(streams_rmsnorm_kernel<AT, N, V>, dim3((unsigned)R), dim3(th), (size_t)(0), st, x, S, y, ldy, mix, out_w, in_w, rows, gain, (AT*)h, W, eps)
+#define GS(AT, V) do { if (S == 1) GO(AT, 1, V); else if (S == 2) GO(AT, 2, V); else if (S == 3) GO(AT, 3, V); else GO(AT, 4, V); } while (0)
+    if (S > 4) { if (act_f32) GO(float, 16, 1); else GO(bf16, 16, 1); }
+    else if (act_f32) { if (vec) GS(float, 4); else GS(float, 1); }
+    else { if (vec) GS(bf16, 4); else GS(bf16, 1); }
+#undef GS
+#undef GO
+    P3_CHECK_LAUNCH("streams_rmsnorm");
     return 0;
 }

@@ -15,7 +15,7 @@ row ends. This engine serves a stream of requests instead:
 
 A model plugs in with kv_layout(), cache_dtype(), prepare(max_context) and forward(StepBatch, pool) (tagenex.TagenexB200), and
 with state_layout() when its layers carry a recurrent state per sequence (dugalix.DugalixB200, danalorn.DanalornB200,
-lupusun.LupusunB200): the pool then keeps one row of fp32 numbers per slot and state buffer, and the step's descriptors list the
+lupusun.LupusunB200, gugezen.GugezenB200): the pool then keeps one row of fp32 numbers per slot and state buffer, and the step's descriptors list the
 sequences of the step (first row, rows, slot, first position) for the kernels that walk a sequence's rows in order.
 """
 import os

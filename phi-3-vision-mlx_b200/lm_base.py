@@ -1,7 +1,7 @@
 """What the engine models (decoders with an fp32 residual stream that run a ragged token batch against the shared page pool) have in
 common: the description of a step, the choice of the matrix-product kernel, the grouped expert products, the attention launches of a
-step and the key-slice cost model of the decode attention. A design (tagenex.py, tapalix.py, dugalix.py, danalorn.py, lupusun.py) owns
-its weights and the order of its kernels; it has no cache and no loop of its own.
+step and the key-slice cost model of the decode attention. A design (tagenex.py, tapalix.py, dugalix.py, danalorn.py, lupusun.py,
+gugezen.py) owns its weights and the order of its kernels; it has no cache and no loop of its own.
 
 Matrix products. Dense bf16 products with K % 8 == 0 run on the tcgen05 GEMM (p3_gemm); batches of at most 16 tokens on the
 weight-streaming kernel (p3_gemm_skinny); everything else (fp32 = true 32-bit on the FMA pipes, grouped expert products, products
@@ -137,12 +137,13 @@ class PagedLM:
         return torch.cat(parts, 0).to(self.dev, self.dtype).contiguous()
 
     # ------------------------------------------------------------------ attention over the page pool
-    def attention_tile_rows(self, H, G, key, val, v_ld):
+    def attention_tile_rows(self, H, G, key, val, v_ld, ld_out=None):
         """query rows per prefill tile that the attention launch takes for these sizes (64: its tensor-core kernels); asked of the
-        library itself so that the engine's tiles and the kernel's choice cannot disagree"""
+        library itself so that the engine's tiles and the kernel's choice cannot disagree. ld_out: pitch of the output rows, when
+        they are wider than the heads"""
         a = _lib.AttnWindowArgs()
         a.q = a.out = a.k_pool = a.v_pool = a.block_table = a.tiles = 256              # aligned stand-ins: nothing is launched
-        a.ld_q, a.ld_out, a.n_heads, a.n_kv, a.dim, a.vdim, a.v_ld = H * key, H * val, H, G, key, val, v_ld
+        a.ld_q, a.ld_out, a.n_heads, a.n_kv, a.dim, a.vdim, a.v_ld = H * key, ld_out or H * val, H, G, key, val, v_ld
         a.act_f32 = a.cache_f32 = self.f32
         return int(_lib.lib().p3_attn_window_tile_rows(C.byref(a)))
 

@@ -129,6 +129,17 @@ def _lupusun_build(cfg, weights, device='cuda', dtype=None, **kw):
     return LupusunB200(cfg, weights, device=device, dtype=dtype or torch.bfloat16)
 
 
+def _gugezen_config(d):
+    from .configs import GugezenConfig
+    return GugezenConfig(d)
+
+
+def _gugezen_build(cfg, weights, device='cuda', dtype=None, **kw):
+    import torch
+    from .gugezen import GugezenB200
+    return GugezenB200(cfg, weights, device=device, dtype=dtype or torch.bfloat16)
+
+
 register('Phi3ForCausalLM', _phi3_config, _phi3_build, 'batch')
 register('Phi3VForCausalLM', _phi3_config, _phi3_build, 'batch')
 register('Tagenex', _tagenex_config, _tagenex_build, 'paged')
@@ -136,3 +147,4 @@ register('Tapalix', _tapalix_config, _tapalix_build, 'paged')
 register('Dugalix', _dugalix_config, _dugalix_build, 'paged')
 register('Danalorn', _danalorn_config, _danalorn_build, 'paged')
 register('Lupusun', _lupusun_config, _lupusun_build, 'paged')
+register('Gugezen', _gugezen_config, _gugezen_build, 'paged')

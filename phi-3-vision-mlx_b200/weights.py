@@ -416,3 +416,80 @@ def random_lupusun_weights(cfg, seed=0, device='cpu'):
             t = rn(shape) / shape[-1] ** 0.5
         w[name] = t.to(torch.bfloat16)
     return w
+
+
+def gugezen_tensor_shapes(cfg):
+    """name -> shape of every tensor of a Gugezen checkpoint; cfg = the config.json dict. A layer that uses another layer's tensors has
+    none of its own."""
+    W, V, S = cfg['width'], cfg['vocab'], int(cfg.get('streams') or 1)
+    out = {'embed': (V, W)}
+    for i, lc in enumerate(cfg['layers']):
+        if lc.get('weights_of') is not None:
+            continue
+        p, m, f = f'l{i}.', lc['mixer'], lc.get('mlp')
+        a = p + 'mix.'
+        if lc['type'] == 'parallel':
+            l, r = m['left'], m['right']
+            H, d, Hr, dr = l['heads'], l['dim'], r['heads'], r['dim']
+            G, dv, dvr = l.get('kv_heads', H), l.get('vdim', d), r.get('vdim', dr)
+            b, c = a + 'left.', a + 'right.'
+            out.update({b + 'q': (H * d, W), b + 'q.b': (H * d,), b + 'k': (G * d, W), b + 'k.b': (G * d,), b + 'v': (G * dv, W),
+                        b + 'v.b': (G * dv,), b + 'sink': (H,), b + 'g': (H * dv, W), b + 'o': (W, H * dv),
+                        c + 'q': (Hr * dr, W), c + 'k': (Hr * dr, W), c + 'v': (Hr * dvr, W), c + 'g': (Hr * dvr, W),
+                        c + 'o': (W, Hr * dvr), c + 'norm': (Hr * dvr,)})
+        elif lc['type'] == 'mamba2':
+            H, N = m['heads'], m['state']
+            inner = H * m['vdim']
+            C = inner + 2 * m.get('groups', 1) * N
+            out.update({a + 'in': (inner + C + H, W), a + 'conv': (C, m['conv']), a + 'conv.b': (C,), a + 'dt_bias': (H,), a + 'A_log': (H,),
+                        a + 'D': (H,), a + 'norm': (inner,), a + 'o': (W, inner)})
+        else:
+            raise NotImplementedError(lc['type'])
+        if f is not None and f['kind'] == 'dense':
+            out.update({p + 'mlp.gate': (f['ff'], W), p + 'mlp.up': (f['ff'], W), p + 'mlp.down': (W, f['ff'])})
+        elif f is not None:
+            units = [(f'e{e}', f['expert']['ff']) for e in range(f['router']['experts'])]
+            units += [('shared', f['shared']['ff'])] if f.get('shared') else []
+            out[p + 'mlp.router'] = (f['router']['experts'], W)
+            for n, ff in units:
+                out.update({f'{p}mlp.{n}.up': (ff, W), f'{p}mlp.{n}.down': (W, ff)})
+        for q in (1, 2) if f is not None else (1,):
+            out.update({f'{p}norm{q}': (W,), f'{p}hc{q}.in': (S,), f'{p}hc{q}.out': (S,), f'{p}hc{q}.mix': (S, S)})
+    out['final.norm'] = (W,)
+    return out
+
+
+def random_gugezen_weights(cfg, seed=0, device='cpu'):
+    """Seeded bf16 tensors for a Gugezen config dict: matrices N(0, 1/fan_in) (router rows twice as large), embedding of unit spread, norm
+    weights around zero, norms of recurrent mixers and skips around one, biases 0.3 N, sinks N(0, 1), convolution taps of spread 0.6;
+    the decays' logarithms and offsets are spread so that heads remember from a few tokens to hundreds. Streams: reads around 1 / S and
+    writes around one, a transfer matrix near the identity whose rows and columns differ."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    rn = lambda s: torch.randn(s, generator=g, device=device, dtype=torch.float32)
+    S = int(cfg.get('streams') or 1)
+    w = {}
+    for name, shape in gugezen_tensor_shapes(cfg).items():
+        leaf = name.split('.', 1)[1] if name.startswith('l') and name[1].isdigit() else name
+        if leaf == 'mix.dt_bias':
+            t = -2.5 + 1.5 * rn(shape)
+        elif leaf == 'mix.A_log':
+            t = 0.5 * rn(shape)
+        elif leaf == 'mix.conv':
+            t = 0.6 * rn(shape)
+        elif leaf.endswith('.b'):
+            t = 0.3 * rn(shape)
+        elif leaf in ('embed', 'mix.left.sink'):
+            t = rn(shape)
+        elif leaf in ('mix.D', 'mix.norm', 'mix.right.norm'):
+            t = 1.0 + 0.1 * rn(shape)
+        elif leaf in ('norm1', 'norm2', 'final.norm'):
+            t = 0.1 * rn(shape)
+        elif leaf.startswith('hc'):
+            t = {'in': lambda: (1.0 + 0.3 * rn(shape)) / S, 'out': lambda: 1.0 + 0.3 * rn(shape),
+                 'mix': lambda: 0.9 * torch.eye(S, device=device) + 0.15 * rn(shape)}[leaf.split('.')[1]]()
+        elif leaf == 'mlp.router':
+            t = 2.0 * rn(shape) / shape[-1] ** 0.5
+        else:
+            t = rn(shape) / shape[-1] ** 0.5
+        w[name] = t.to(torch.bfloat16)
+    return w
