@@ -891,6 +891,81 @@ def run_lupusun(args):
           'steps': args.steps, 'warmup': max(3, args.warmup), 'peaks': {'hbm_gbs': hbm, 'bf16_tflops': tf}, 'sizes': out})
 
 
+# ------------------------------------------------------------------------------------------------ --arch gugezen
+def _gugezen_cfg(width, heads, kv, dim, mh, mdim, mvdim, sh, svdim, state, groups, parts, ff, eff, experts, top, shared, streams, layers, vocab):
+    par = {'type': 'parallel',
+           'mixer': {'left': {'heads': heads, 'kv_heads': kv, 'dim': dim, 'vdim': dim, 'scale': dim ** -0.5,
+                              'rot': {'base': 500000.0, 'dims': dim, 'scaling': {'factor': 8.0, 'low': 1.0, 'high': 4.0, 'original': 8192}}},
+                     'right': {'heads': mh, 'dim': mdim, 'vdim': mvdim, 'decay': [1.0 - 2.0 ** -(4 + 0.5 * h) for h in range(mh)]},
+                     'left_scale': 0.7, 'right_scale': 0.7}}
+    ssm = {'type': 'mamba2', 'mixer': {'heads': sh, 'vdim': svdim, 'state': state, 'groups': groups, 'conv': 4, 'norm_groups': parts}}
+    dense = {'kind': 'dense', 'ff': ff}
+    moe = {'kind': 'moe', 'expert': {'ff': eff}, 'router': {'experts': experts, 'top': top}, 'shared': {'ff': shared}}
+    return {'architecture': 'Gugezen', 'vocab': vocab, 'width': width, 'norm': {'eps': 1e-5}, 'embedding': {'scale': 1.0}, 'streams': streams,
+            'logit_scale': 1.0, 'layers': [dict(ssm if i % 2 else par, mlp=(moe if i % 2 else dense)) for i in range(layers)]}
+
+
+def run_gugezen(args):
+    """Throughput of the Gugezen design on the continuous-batching engine at layer sizes of a real model (random weights, bf16 serving
+    mode), beside the two closest existing models (same engine, page pool with state rows, product and attention kernels) at equal width
+    and depth: Dugalix (attention beside a recurrence in one layer, softmax router with a shared unit) with the same attention shape,
+    recurrent state shape and expert sizes, and Lupusun (convolutions in front of a recurrence, gated units) with the same number of
+    state numbers and convolved channels. One JSON line: per size the prefill and decode tok/s of all and, per kernel family, time and
+    achieved FLOP/s (prefill) or bytes/s (decode) against the measured peaks."""
+    import torch
+    import phi3_b200  # noqa: F401
+    from phi3_b200 import weights
+    from phi3_b200.dugalix import DugalixB200
+    from phi3_b200.gugezen import GugezenB200
+    from phi3_b200.lupusun import LupusunB200
+    hbm, _ = peaks()
+    tf = json.load(open(os.path.join(ROOT, 'MEASURED_PEAKS.json'))).get('bf16_tflops', 1590.0) if os.path.exists(
+        os.path.join(ROOT, 'MEASURED_PEAKS.json')) else 1590.0
+    dev = torch.device('cuda:0')
+    a = dict(width=2048, heads=16, kv=4, dim=128, mh=8, mdim=128, mvdim=256, sh=64, svdim=64, state=128, groups=8, parts=8, ff=8192, eff=1408,
+             experts=8, top=2, shared=2816, streams=2, layers=4)
+    c = dict(width=3072, heads=32, kv=8, dim=64, mh=12, mdim=64, mvdim=256, sh=48, svdim=128, state=64, groups=1, parts=1, ff=8192, eff=1024,
+             experts=16, top=4, shared=2048, streams=4, layers=4)
+    sizes = [dict(a, name='w2048_h16x128_kv4_m8x128x256_s64x128x64_e8x1408_r2_L4'),
+             dict(a, name='w2048_h16x128_kv4_m8x128x256_s64x128x64_e8x1408_r2_L4_b16', batch=16),
+             dict(c, name='w3072_h32x64_kv8_m12x64x256_s48x64x128_e16x1024_r4_L4')]
+    if getattr(args, 'sizes', None):
+        sizes = [sz for i, sz in enumerate(sizes) if str(i) in args.sizes.split(',')]
+    vocab, L, CTX_D, NEW_D = 32064, 2048, 2048, 32
+    out = []
+    for sz in sizes:
+        B, name = sz.pop('batch', 4), sz.pop('name')
+        row = dict(size=name, batch=B, prompt=L)
+
+        def measure(key, cls, cfg, init):
+            m = cls(cfg, init(cfg, 0, device=dev), dtype=torch.bfloat16)
+            _, row[key] = _engine_model_numbers(m, B, L, CTX_D, NEW_D, vocab, args, hbm, tf)
+            del m
+            torch.cuda.empty_cache()
+
+        measure('gugezen', GugezenB200, _gugezen_cfg(vocab=vocab, **sz), weights.random_gugezen_weights)
+        # Dugalix: parallel layers throughout (no window), mixtures and dense units alternate as above, no identity experts, no groups
+        par = {'type': 'parallel',
+               'mixer': {'left': {'heads': sz['heads'], 'kv_heads': sz['kv'], 'dim': sz['dim'], 'vdim': sz['dim'], 'scale': sz['dim'] ** -0.5,
+                                  'rot': {'base': 500000.0, 'dims': sz['dim']}},
+                         'right': {'heads': sz['mh'], 'dim': sz['mdim'], 'vdim': sz['mvdim'], 'gate_cap': 15.0}, 'left_scale': 0.7, 'right_scale': 0.7}}
+        dense = {'kind': 'dense', 'ff': sz['ff']}
+        moe = {'kind': 'moe', 'expert': {'ff': sz['eff']}, 'router': {'experts': sz['experts'], 'top': sz['top']}, 'shared': {'ff': sz['shared']}}
+        measure('dugalix_equal_size', DugalixB200,
+                {'architecture': 'Dugalix', 'vocab': vocab, 'width': sz['width'], 'norm': {'eps': 1e-5}, 'residual_mult': 0.6,
+                 'layers': [dict(par, mlp=(moe if i % 2 else dense)) for i in range(sz['layers'])]}, weights.random_dugalix_weights)
+        # Lupusun: its recurrence with the state-space layer's heads, groups and sizes, its attention with the parallel layer's shape
+        att = {'type': 'attention', 'mixer': {'heads': sz['heads'], 'kv_heads': sz['kv'], 'dim': sz['dim'], 'vdim': sz['dim'], 'scale': sz['dim'] ** -0.5,
+                                              'rot': {'base': 500000.0, 'dims': sz['dim']}}}
+        delta = {'type': 'delta', 'mixer': {'heads': sz['sh'], 'kv_heads': sz['groups'], 'dim': sz['state'], 'vdim': sz['svdim'], 'conv': 4}}
+        measure('lupusun_equal_size', LupusunB200,
+                {'architecture': 'Lupusun', 'vocab': vocab, 'width': sz['width'], 'norm': {'eps': 1e-5}, 'residual_mult': 0.9,
+                 'layers': [dict(delta if i % 2 else att, mlp=dense) for i in range(sz['layers'])]}, weights.random_lupusun_weights)
+        out.append(row)
+    _emit({"metric": "gugezen_prefill_decode_tok_per_s", 'arch': 'gugezen', 'dtype': 'bf16', 'data': 'synthetic', 'n_gpus': 1,
+          'steps': args.steps, 'warmup': max(3, args.warmup), 'peaks': {'hbm_gbs': hbm, 'bf16_tflops': tf}, 'sizes': out})
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument('--gpus', type=int, default=1)
@@ -898,10 +973,10 @@ def main():
     ap.add_argument('--warmup', type=int, default=3)
     ap.add_argument('--impl', default='b200', choices=['b200', 'reference'])
     ap.add_argument('--no-cpu-baseline', action='store_true')
-    ap.add_argument('--arch', default='phi3', choices=['phi3', 'tagenex', 'tapalix', 'dugalix', 'danalorn', 'lupusun'],
-                    help='phi3: the headline workload (default); tagenex / tapalix / dugalix / danalorn / lupusun: prefill / decode throughput of '
+    ap.add_argument('--arch', default='phi3', choices=['phi3', 'tagenex', 'tapalix', 'dugalix', 'danalorn', 'lupusun', 'gugezen'],
+                    help='phi3: the headline workload (default); tagenex / tapalix / dugalix / danalorn / lupusun / gugezen: prefill / decode throughput of '
                          'that design on the continuous-batching engine, beside the closest existing model at equal size')
-    ap.add_argument('--sizes', default='', help='with --arch dugalix / danalorn / lupusun: indices of the sizes to run, with commas (default: all)')
+    ap.add_argument('--sizes', default='', help='with --arch dugalix / danalorn / lupusun / gugezen: indices of the sizes to run, with commas (default: all)')
     args = ap.parse_args()
     if not (args.gpus > 1 and int(os.environ.get('WORLD_SIZE', 1)) == 1):      # the self-launching parent just relays its child
         _claim_stdout()
@@ -917,6 +992,8 @@ def main():
         return run_danalorn(args)
     if args.arch == 'lupusun':
         return run_lupusun(args)
+    if args.arch == 'gugezen':
+        return run_gugezen(args)
     world = int(os.environ.get('WORLD_SIZE', 1))
     if args.gpus > 1 and world == 1:
         # convenience: self-launch under torchrun when called directly with --gpus N

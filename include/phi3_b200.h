@@ -525,7 +525,8 @@ int p3_router_groups(const float* logits, int64_t ld_logits, const float* correc
                      float scale, int mode, int32_t* ids, float* wts, cudaStream_t st);
 
 /* out[t] = sum_j wts[t][j] * (ids[t][j] < n_real ? y[where[t * top + j]] : h[t]) + (add ? add[t] : 0): experts with an index of
- * n_real or more are identity experts, whose output is the layer's input h (fp32 [T, W]); add fp32 [T, ld_add] or NULL */
+ * n_real or more are identity experts, whose output is the layer's input h (fp32 [T, W]); ids NULL: there are none (h is not read); add
+ * fp32 [T, ld_add] or NULL */
 int p3_moe_combine_identity(const float* y, int64_t ldy, const int32_t* where, const int32_t* ids, const float* wts, int top,
                             int n_real, const float* h, const float* add, int64_t ld_add, float* out, int64_t T, int W,
                             cudaStream_t st);

@@ -344,6 +344,17 @@ __global__ void gather_rows_kernel(const AT* __restrict__ x, int64_t ldx, const 
     for (int i = threadIdx.x; i < W; i += blockDim.x) out[(size_t)r * W + i] = src[i];
 }
 
+// rows of whole 16-byte vectors (n16 per row)
+__global__ void gather_rows_vec_kernel(const uint4* __restrict__ x, int64_t ldx16, const int32_t* __restrict__ rows, int div,
+                                       uint4* __restrict__ out, int n16) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    const int64_t r = blockIdx.x;
+    const uint4* src = x + (size_t)(rows[r] / div) * ldx16;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < n16; i += blockDim.x) out[(size_t)r * n16 + i] = src[i];
+}
+
 // ---------------------------------------------------------------- out[t] = sum_j w[t][j] * y[where[t * top + j]]   (j ascending)
 __global__ void moe_combine_kernel(const float* __restrict__ y, int64_t ldy, const int32_t* __restrict__ where,
                                    const float* __restrict__ wts, int top, float* __restrict__ out, int W) {
@@ -953,7 +964,7 @@ __global__ void moe_combine_identity_kernel(const float* __restrict__ y, int64_t
     const int64_t t = blockIdx.x;
     for (int j = threadIdx.x; j < top; j += blockDim.x) {
         cw[j] = wts[t * top + j];
-        rows[j] = ids[t * top + j] < n_real ? where[t * top + j] : -1;
+        rows[j] = !ids || ids[t * top + j] < n_real ? where[t * top + j] : -1;
     }
     __syncthreads();
     for (int i = threadIdx.x; i < W; i += blockDim.x) {
@@ -962,6 +973,29 @@ __global__ void moe_combine_identity_kernel(const float* __restrict__ y, int64_t
 #pragma unroll 4
         for (int j = 0; j < top; j++) s = fmaf(cw[j], rows[j] >= 0 ? y[(size_t)rows[j] * ldy + i] : hv, s);
         out[(size_t)t * W + i] = s + (add ? add[(size_t)t * ld_add + i] : 0.f);
+    }
+}
+
+// the same without identity experts, four columns per thread (W and the pitches multiples of four, 16-byte aligned rows)
+__global__ void moe_combine_vec4_kernel(const float* __restrict__ y, int64_t ldy, const int32_t* __restrict__ where,
+                                        const float* __restrict__ wts, int top, const float* __restrict__ add, int64_t ld_add,
+                                        float* __restrict__ out, int W) {
+    pdl_trigger();                                           // the next kernel may set up while this one runs ...
+    pdl_wait();                                              // ... and this one touches memory only after its predecessors are done
+    const int64_t t = blockIdx.x;
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int j = 0; j < top; j++) {
+            const float w = wts[t * top + j];
+            const float4 v = *reinterpret_cast<const float4*>(y + (size_t)where[t * top + j] * ldy + i);
+            s.x = fmaf(w, v.x, s.x); s.y = fmaf(w, v.y, s.y); s.z = fmaf(w, v.z, s.z); s.w = fmaf(w, v.w, s.w);
+        }
+        if (add) {
+            const float4 v = *reinterpret_cast<const float4*>(add + (size_t)t * ld_add + i);
+            s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+        }
+        *reinterpret_cast<float4*>(out + (size_t)t * W + i) = s;
     }
 }
 // ---------------------------------------------------------------- embedding plus the row of a hashed (previous, current) token pair
@@ -1402,15 +1436,31 @@ extern "C" int p3_gather_rows(const void* x, int64_t ldx, int x_f32, const int32
                               cudaStream_t st) {
     P3_CHECK_ARG(div >= 1 && rows, "gather_rows: need an index list and div >= 1");
     if (R == 0) return 0;
+    const int per16 = x_f32 ? 4 : 8;                         // numbers per 16 bytes
+    if (W % per16 == 0 && ldx % per16 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
+        const int n16 = W / per16;
+        p3_launch_pdl(gather_rows_vec_kernel, dim3((unsigned)R), dim3(n16 >= 256 ? 128 : 64), (size_t)(0), st, (const uint4*)x, ldx / per16, rows, div, (uint4*)out, n16);
+        P3_CHECK_LAUNCH("gather_rows");
+        return 0;
+    }
     if (x_f32) p3_launch_pdl(gather_rows_kernel<float>, dim3((unsigned)R), dim3(128), (size_t)(0), st, (const float*)x, ldx, rows, div, (float*)out, W);
     else p3_launch_pdl(gather_rows_kernel<bf16>, dim3((unsigned)R), dim3(128), (size_t)(0), st, (const bf16*)x, ldx, rows, div, (bf16*)out, W);
     P3_CHECK_LAUNCH("gather_rows");
     return 0;
 }
 
+static bool combine_vec_ok(const float* y, int64_t ldy, const float* add, int64_t ld_add, const float* out, int W) {
+    return W % 4 == 0 && ldy % 4 == 0 && (!add || ld_add % 4 == 0) && (((uintptr_t)y | (uintptr_t)add | (uintptr_t)out) & 15) == 0;
+}
+
 extern "C" int p3_moe_combine(const float* y, int64_t ldy, const int32_t* where, const float* wts, int top, float* out, int64_t T, int W,
                               cudaStream_t st) {
     if (T == 0) return 0;
+    if (combine_vec_ok(y, ldy, nullptr, 0, out, W)) {
+        p3_launch_pdl(moe_combine_vec4_kernel, dim3((unsigned)T), dim3(W >= 1024 ? 256 : 64), (size_t)(0), st, y, ldy, where, wts, top, (const float*)nullptr, (int64_t)0, out, W);
+        P3_CHECK_LAUNCH("moe_combine");
+        return 0;
+    }
     p3_launch_pdl(moe_combine_kernel, dim3((unsigned)T), dim3(W >= 1024 ? 256 : 128), (size_t)((size_t)top * 8), st, y, ldy, where, wts, top, out, W);
     P3_CHECK_LAUNCH("moe_combine");
     return 0;
@@ -1608,8 +1658,13 @@ extern "C" int p3_relu2(const float* u, int64_t ld, const float* row_gate, int64
 extern "C" int p3_moe_combine_identity(const float* y, int64_t ldy, const int32_t* where, const int32_t* ids, const float* wts, int top,
                                        int n_real, const float* h, const float* add, int64_t ld_add, float* out, int64_t T, int W,
                                        cudaStream_t st) {
-    P3_CHECK_ARG(y && where && ids && wts && out, "moe_combine_identity: null argument");
+    P3_CHECK_ARG(y && where && wts && out, "moe_combine_identity: null argument");
     if (T == 0) return 0;
+    if (!ids && combine_vec_ok(y, ldy, add, ld_add, out, W)) {
+        p3_launch_pdl(moe_combine_vec4_kernel, dim3((unsigned)T), dim3(W >= 1024 ? 256 : 64), (size_t)(0), st, y, ldy, where, wts, top, add, ld_add, out, W);
+        P3_CHECK_LAUNCH("moe_combine_identity");
+        return 0;
+    }
     p3_launch_pdl(moe_combine_identity_kernel, dim3((unsigned)T), dim3(W >= 1024 ? 256 : 128), (size_t)(2 * top * sizeof(float)), st,
                   y, ldy, where, ids, wts, top, n_real, h, add, ld_add, out, W);
     P3_CHECK_LAUNCH("moe_combine_identity");

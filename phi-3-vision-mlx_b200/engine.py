@@ -82,9 +82,9 @@ class Engine:
             raise PoolExhausted(f'page pool exhausted: the step wants {need} pages, {len(pool.free_pages)} of {pool.n_pages} free')
         if self.stateful and any(n > 1 for n in (sum(1 for r, t, _ in entries if r == rid and len(t)) for rid in grow)):
             raise ValueError('a request may bring its tokens of a step in one entry only: its recurrent state advances once per step')
-        ids, slots, poss, pf, dec, want, seqs = [], [], [], [], [], [], []
+        ids, slots, poss, pf, dec, want, seqs = [], [], [], [], [], [], []     # numpy pieces / records, in entry order
         slot_seq = [0] * pool.n_slots                        # slot -> its record in seqs (slots without tokens are never looked up)
-        row = 0
+        row = max_pos = 0
         for rid, toks, wanted in entries:
             n = len(toks)
             if n == 0:
@@ -93,16 +93,17 @@ class Engine:
                 self.slot_of[rid] = pool.admit()
             s = self.slot_of[rid]
             p0 = pool.extend(s, n)
-            ids.extend(int(t) for t in toks)
-            slots.extend([s] * n)
-            poss.extend(range(p0, p0 + n))
+            ids.append(np.asarray(toks, np.int32))
+            slots.append(np.full(n, s, np.int32))
+            poss.append(np.arange(p0, p0 + n, dtype=np.int32))
+            max_pos = max(max_pos, p0 + n - 1)
             slot_seq[s] = len(seqs)
             seqs.append((row, n, s, p0))
             if n == 1:
                 dec.append((row, 1, s, p0))
             else:
-                for r0 in range(0, n, self.q_tile):
-                    pf.append((row + r0, min(self.q_tile, n - r0), s, p0 + r0))
+                r0 = np.arange(0, n, self.q_tile, dtype=np.int32)
+                pf.append(np.stack([row + r0, np.minimum(self.q_tile, n - r0), np.full_like(r0, s), p0 + r0], 1))
             for i in wanted:
                 if not 0 <= i < n:
                     raise IndexError(f'request {rid}: wanted index {i} outside its {n} tokens')
@@ -110,17 +111,16 @@ class Engine:
             row += n
         T = row
         b = StepBatch()
-        b.T, b.n_pf, b.n_dec, b.R, b.n_seq, b.n_slots = T, len(pf), len(dec), len(want), len(seqs), pool.n_slots
-        b.max_pos = max(poss) if poss else 0
+        b.T, b.n_pf, b.n_dec, b.R, b.n_seq, b.n_slots = T, sum(len(p) for p in pf), len(dec), len(want), len(seqs), pool.n_slots
+        b.max_pos = max_pos
         if T == 0:
             return b
-        flat = np.concatenate([np.asarray(ids, np.int32), np.asarray(slots, np.int32), np.asarray(poss, np.int32),
-                               np.asarray(pf, np.int32).reshape(-1), np.asarray(dec, np.int32).reshape(-1),
-                               np.asarray(seqs, np.int32).reshape(-1), np.asarray(want, np.int32),
-                               np.asarray(slot_seq, np.int32)])
-        pad = (-3 * T) % 4                                   # tile records are read as 16-byte vectors
-        flat = np.concatenate([flat[:3 * T], np.zeros(pad, np.int32), flat[3 * T:]])
-        d = torch.from_numpy(flat).to(self.dev)
+        i32 = lambda v: np.asarray(v, np.int32).reshape(-1)
+        pad = np.zeros((-3 * T) % 4, np.int32)               # tile records are read as 16-byte vectors
+        flat = torch.from_numpy(np.concatenate(ids + slots + poss + [pad] + [p.reshape(-1) for p in pf] +
+                                               [i32(dec), i32(seqs), i32(want), i32(slot_seq)]))
+        # from pinned memory the upload is asynchronous: the host goes on launching (or preparing the next step) meanwhile
+        d = flat.pin_memory().to(self.dev, non_blocking=True) if self.dev.type == 'cuda' else flat.to(self.dev)
         self._bind(b, d)
         pool.sync()
         return b

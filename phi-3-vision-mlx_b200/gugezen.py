@@ -36,7 +36,7 @@ import os
 
 import torch
 from . import _lib
-from ._lib import call, call_struct, ptr
+from ._lib import call_struct, ptr
 from .configs import GugezenConfig, wavelength_frequencies
 from .lm_base import PagedLM, _stream
 
@@ -204,11 +204,11 @@ class GugezenB200(PagedLM):
         f = L['cfg'].ff
         return None if f is None else L['gu'] if f.kind == 'dense' else L['in2_w']
 
-    def _scan(self, s, L, state, b, T, H, d, dv, nbytes):
+    def _scan(self, kind, s, state, b, T, H, d, dv, nbytes):
         s.n_heads, s.dim, s.vdim, s.state, s.seqs, s.n_seqs = H, d, dv, ptr(state), ptr(b.seqs), b.n_seq
         ev = self._ev()
         call_struct('p3_decay_scan', s, _stream())
-        self._ev(ev, 'decay_scan', 4 * T * H * d * dv, b.n_seq * H * d * dv * 8 + nbytes)
+        self._ev(ev, kind, 4 * T * H * d * dv, b.n_seq * H * d * dv * 8 + nbytes)
 
     def _parallel(self, L, li, h, b, pool):
         """normed input h (act [T, W]) -> mixer output, fp32 [T, W]"""
@@ -237,7 +237,7 @@ class GugezenB200(PagedLM):
             s.qkv, s.ld_qkv, s.n_kv, s.decay = ptr(proj), proj.stride(0), Hm, ptr(L['decay'])
             s.q_off, s.k_off, s.v_off = L['m_off'], L['m_off'] + Hm * dm, L['m_off'] + 2 * Hm * dm
             s.out, s.ld_out = ptr(o), o.stride(0)
-            self._scan(s, L, pool.state[self._state_of[li]], b, T, Hm, dm, dvm, T * (2 * Hm * dm + 2 * n_mem) * 4)
+            self._scan('memory_scan', s, pool.state[self._state_of[li]], b, T, Hm, dm, dvm, T * (2 * Hm * dm + 2 * n_mem) * 4)
             self.rows('headnorm', T * n_mem * (8 + esz), 'p3_part_norm_gate', ptr(o), o.stride(0), 1, n_mem, ptr(L['m_gain']),
                       ptr(proj[:, L['mg_off']:]), proj.stride(0), 0, 0, m.mem_scale, self.eps, ptr(cat[:, n_att:]), cat.stride(0), self.f32, T, _stream())
 
@@ -287,7 +287,7 @@ class GugezenB200(PagedLM):
         s.qkv, s.ld_qkv, s.v_off, s.k_off, s.q_off = ptr(xbc), xbc.stride(0), 0, inner, inner + G * N
         s.n_kv, s.gates, s.skip, s.out, s.ld_out = G, ptr(gates), ptr(L['skip']), ptr(o), o.stride(0)
         s.conv_in, s.ld_conv_in, s.channels, s.taps, s.conv_state = ptr(proj[:, inner:]), proj.stride(0), C, m.taps, ptr(history)
-        self._scan(s, L, state, b, T, H, N, dv, T * (C + inner) * 4)
+        self._scan('ssm_scan', s, state, b, T, H, N, dv, T * (C + inner) * 4)
         cat = e(T, inner, dt=self.dtype)
         self.rows('headnorm', T * inner * (8 + (4 if self.f32 else 2)), 'p3_part_norm_gate', ptr(o), o.stride(0), m.norm_groups,
                   inner // m.norm_groups, ptr(L['m_gain']), ptr(proj), proj.stride(0), 1, 1, 1.0, self.eps, ptr(cat), cat.stride(0), self.f32, T, st)
@@ -316,15 +316,18 @@ class GugezenB200(PagedLM):
         e = lambda *s, dt=torch.float32: torch.empty(s, dtype=dt, device=self.dev)
         p2 = e(T, L['in2_w'].shape[0])
         self.linear(h, L['in2_w'], p2, nxt=L['sh_down'])
-        ysh = None
-        if f.shared_ff:
-            shid, ysh = e(T, f.shared_ff, dt=self.dtype), e(T, W)
+        shid, ysh = (e(T, f.shared_ff, dt=self.dtype), e(T, W)) if f.shared_ff else (None, None)
+
+        def shared():
             self._gelu(p2, shid, T, f.shared_ff)
             self.linear(shid, L['sh_down'], ysh)
+
         ids, wts, y = e(T, f.top, dt=torch.int32), e(T, f.top), e(T, W)
-        call('p3_router_groups', ptr(p2[:, f.shared_ff:]), p2.stride(0), None, T, f.experts, f.top, 1, 1, 1.0, _lib.ROUTER_SOFTMAX, ptr(ids),
-             ptr(wts), st)
-        combine = lambda dn, where: call('p3_moe_combine_identity', ptr(dn), dn.stride(0), ptr(where), ptr(ids), ptr(wts), f.top, f.experts,
-                                         None, ptr(ysh), ysh.stride(0) if ysh is not None else 0, ptr(y), T, W, st)
-        self.experts(L['up'], L['down'], f, h, y, T, ids, wts, lambda up, hid, n: self._gelu(up, hid, n, f.ff), combine=combine)
+        self.rows('route', T * (f.experts * 4 + f.top * 8), 'p3_router_groups', ptr(p2[:, f.shared_ff:]), p2.stride(0), None, T, f.experts,
+                  f.top, 1, 1, 1.0, _lib.ROUTER_SOFTMAX, ptr(ids), ptr(wts), st)
+        nb = T * W * 4 * (f.top + (1 if ysh is None else 2))
+        combine = lambda dn, where: self.rows('combine', nb, 'p3_moe_combine_identity', ptr(dn), dn.stride(0), ptr(where), None, ptr(wts), f.top,
+                                              f.experts, None, ptr(ysh), ysh.stride(0) if ysh is not None else 0, ptr(y), T, W, st)
+        self.experts(L['up'], L['down'], f, h, y, T, ids, wts, lambda up, hid, n: self._gelu(up, hid, n, f.ff), combine=combine,
+                     meanwhile=shared if f.shared_ff else None)
         return y

@@ -178,32 +178,41 @@ class PagedLM:
             self._ev(ev, 'attn_decode', 2 * b.n_dec * H * span * (key + val), b.n_dec * span * kv_bytes * esz)
 
     # ------------------------------------------------------------------ mixture of experts behind a router
-    def experts(self, gu_w, down_w, f, xa, y, T, ids, wts, glu, n_sorted=None, combine=None):
+    def experts(self, gu_w, down_w, f, xa, y, T, ids, wts, glu, n_sorted=None, combine=None, meanwhile=None):
         """ids / wts [T, top] from the design's router -> y fp32 [T, W] = sum of the chosen experts' outputs. gu_w [E, 2 ff, W] holds
         every expert's gate rows over its up rows, down_w [E, W, ff]; glu(gu fp32 [n, 2 ff], hid act [n, ff], n) is the design's
         activation. The (token, choice) pairs are sorted by expert and run as two grouped products over the sorted rows.
         A unit without a gate passes its up matrices alone ([E, ff, W]; the activation then gets [n, ff]). n_sorted: the router
         scores this many outputs, of which only the first f.experts have matrices (the pairs of the others are sorted behind them
-        and skipped by the products); combine(dn, where) then replaces the plain weighted sum."""
+        and skipped by the products); combine(dn, where) then replaces the plain weighted sum. meanwhile(): work that does not
+        depend on the choice (a shared unit); launched so that it covers the wait for the segment offsets."""
         st, dev, n = _stream(), self.dev, T * f.top
         n_sorted = f.experts if n_sorted is None else n_sorted
         up = gu_w.shape[1]
         seg = torch.empty(n_sorted + 1, dtype=torch.int32, device=dev)
         order = torch.empty(n, dtype=torch.int32, device=dev)
         where = torch.empty(n, dtype=torch.int32, device=dev)
-        call('p3_moe_sort', ptr(ids), n, n_sorted, ptr(seg), ptr(order), ptr(where), st)
+        self.rows('route', n * 12, 'p3_moe_sort', ptr(ids), n, n_sorted, ptr(seg), ptr(order), ptr(where), st)
         gu = torch.empty((n, up), dtype=torch.float32, device=dev)
         hid = torch.empty((n, f.ff), dtype=self.dtype, device=dev)
         dn = torch.empty((n, self.W), dtype=torch.float32, device=dev)
-        # Large batches (prompt portions): the segment offsets are read back (one small D2H per mixture layer) and every expert's
-        # rows go through the tcgen05 GEMM as a dense product over the gathered, expert-ordered activations. Small batches stay
-        # on the device-side grouped kernel, which needs no host knowledge of the counts.
+        # Large batches (prompt portions): the segment offsets are read back (one small D2H per mixture layer, behind which the gather
+        # and `meanwhile` keep the device busy) and every expert's rows go through the tcgen05 GEMM as a dense product over the gathered,
+        # expert-ordered activations. Small batches stay on the device-side grouped kernel, which needs no host knowledge of the counts.
         dense = self.experts_dense(f, T)
+        if dense:
+            cut = torch.empty(n_sorted + 1, dtype=torch.int32, pin_memory=True)
+            cut.copy_(seg, non_blocking=True)
+            landed = torch.cuda.Event()
+            landed.record()
+        if meanwhile is not None:
+            meanwhile()
         ev = self._ev()
         if dense:
             xs = torch.empty((n, self.W), dtype=self.dtype, device=dev)
             call('p3_gather_rows', ptr(xa), xa.stride(0), self.f32, ptr(order), f.top, ptr(xs), n, self.W, st)
-            cut = seg.tolist()
+            landed.synchronize()
+            cut = cut.tolist()
             for ex in range(f.experts):
                 a0, a1 = cut[ex], cut[ex + 1]
                 if a1 > a0:
@@ -226,7 +235,8 @@ class PagedLM:
         if combine is not None:
             combine(dn, where)
         else:
-            call('p3_moe_combine', ptr(dn), dn.stride(0), ptr(where), ptr(wts), f.top, ptr(y), T, self.W, st)
+            self.rows('combine', T * self.W * 4 * (f.top + 1), 'p3_moe_combine', ptr(dn), dn.stride(0), ptr(where), ptr(wts), f.top, ptr(y), T,
+                      self.W, st)
 
     def experts_dense(self, f, T):
         """do the experts of a step with T tokens run as dense per-expert products (which reads the segment offsets back)?"""

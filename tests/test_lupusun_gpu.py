@@ -748,7 +748,7 @@ def test_gated_units_with_both_activations(lib):
                 torch.cuda.synchronize()
                 assert (out.float().cpu() - fn(gu[:, :F]) * gu[:, F:]).abs().max() < (1e-5 if dt == F32 else 3e-2)
     with pytest.raises(RuntimeError):
-        call('p3_glu_act', ptr(gd), ptr(gd), 33, ptr(gd), 33, 1, 1, 33, 2, 0)
+        call('p3_glu_act', ptr(gd), ptr(gd), 33, ptr(gd), 33, 1, 1, 33, 9, 0)
 
 
 # ------------------------------------------------------------------------------------------------ entry points
