@@ -52,7 +52,7 @@
 // Duality": q = C, k = B, v = x, g = exp(-exp(A) dt), b = dt, heads in groups that share B and C, a skip factor c) and, with a constant
 // g per head, b = 1 and c = 0, linear attention with fixed decays.
 //   short_conv_kernel           as above, with a bias per channel; the gates are then g and b = dt
-//   delta_scan_kernel           with DELTA = false: one pass over the state columns per token
+//   delta_scan_kernel           with DELTA = false: one pass over the state columns per token, four tokens between two reductions
 //   part_norm_gate_kernel       rows normed in equal parts (one part: all heads together), with the gate in front of the norm or behind it
 #include "common.cuh"
 #include "../../include/phi3_b200.h"
@@ -648,8 +648,57 @@ __global__ void __launch_bounds__(GLA_WARPS * 32) delta_scan_kernel(p3_delta_sca
         const float* ks = qs + TB * DPP;
         const float* vs = ks + TB * DPP;
         const float* gs = vs + TB * COLS;
+        int tt = 0;
+        if constexpr (!DELTA && DS <= 64) {
+            // four tokens at a time: no sum of one of them waits for another's shuffles, and the row slices share the reduction out, so
+            // that slice s ends with the whole sums of token s (RS = 4; of tokens s and s + 2 with RS = 2) and writes them
+            for (; tt + 4 <= nb; tt += 4) {
+                float p[4][NC];
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    const float keep = a.gates ? gs[2 * (tt + i)] : fixed, beta = a.gates ? gs[2 * (tt + i) + 1] : 1.f;
+                    const float4* kq = reinterpret_cast<const float4*>(ks + (tt + i) * DPP + at_row(d0));
+                    const float4* qq = reinterpret_cast<const float4*>(qs + (tt + i) * DPP + at_row(d0));
+                    float acc[NC][4], u[NC];
+#pragma unroll
+                    for (int c = 0; c < NC; c++) {
+                        acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
+                        u[c] = beta * vs[(tt + i) * COLS + warp * WCOLS + lane % CW + c * CW];
+                    }
+#pragma unroll
+                    for (int j = 0; j < DS; j += 4) {
+                        const float4 kk = kq[j / 4], qv = qq[j / 4];
+#pragma unroll
+                        for (int c = 0; c < NC; c++) {
+                            S[c][j] = fmaf(kk.x, u[c], keep * S[c][j]);         acc[c][0] = fmaf(S[c][j], qv.x, acc[c][0]);
+                            S[c][j + 1] = fmaf(kk.y, u[c], keep * S[c][j + 1]); acc[c][1] = fmaf(S[c][j + 1], qv.y, acc[c][1]);
+                            S[c][j + 2] = fmaf(kk.z, u[c], keep * S[c][j + 2]); acc[c][2] = fmaf(S[c][j + 2], qv.z, acc[c][2]);
+                            S[c][j + 3] = fmaf(kk.w, u[c], keep * S[c][j + 3]); acc[c][3] = fmaf(S[c][j + 3], qv.w, acc[c][3]);
+                        }
+                    }
+#pragma unroll
+                    for (int c = 0; c < NC; c++) p[i][c] = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
+                }
+                const int sl = lane / CW;
+                float r[2][NC];
+#pragma unroll
+                for (int h = 0; h < 2; h++)
+#pragma unroll
+                    for (int c = 0; c < NC; c++)
+                        r[h][c] = (sl & 1 ? p[2 * h + 1][c] : p[2 * h][c]) + __shfl_xor_sync(0xffffffffu, sl & 1 ? p[2 * h][c] : p[2 * h + 1][c], CW);
+                auto write = [&](int t, int c, float y) {
+                    y = fmaf(skip, vs[t * COLS + warp * WCOLS + lane % CW + c * CW], y);
+                    if (col + c * CW < dv) a.out[(size_t)(row0 + t0 + t) * a.ld_out + (size_t)hd * dv + col + c * CW] = y;
+                };
+#pragma unroll
+                for (int c = 0; c < NC; c++) {
+                    if (RS == 4) write(tt + sl, c, (sl & 2 ? r[1][c] : r[0][c]) + __shfl_xor_sync(0xffffffffu, sl & 2 ? r[0][c] : r[1][c], 2 * CW));
+                    else { write(tt + sl, c, r[0][c]); write(tt + 2 + sl, c, r[1][c]); }
+                }
+            }
+        }
 #pragma unroll(DS >= (DELTA ? 64 : 128) ? 1 : 2)
-        for (int tt = 0; tt < nb; tt++) {
+        for (; tt < nb; tt++) {
             const float keep = DELTA || a.gates ? gs[2 * tt] : fixed, beta = DELTA || a.gates ? gs[2 * tt + 1] : 1.f;
             const float4* kq = reinterpret_cast<const float4*>(ks + tt * DPP + at_row(d0));
             const float4* qq = reinterpret_cast<const float4*>(qs + tt * DPP + at_row(d0));
@@ -985,8 +1034,10 @@ int launch_scan(const p3_delta_scan_args* a, cudaStream_t st, const char* who) {
     P3_CHECK_ARG(a->taps <= 1 || (a->conv_in && a->conv_state && a->channels >= 1), "%s: the convolution history needs its inputs", who);
     P3_CHECK_ARG(((uintptr_t)a->seqs & 15) == 0, "%s: the sequence records must be 16-byte aligned", who);
     if (a->n_seqs == 0) return 0;
-    // A warp is four row slices x eight lanes, a lane owns one or two columns: the choice of the linear-attention scan
-    int rs = 4, nc = (int64_t)a->n_seqs * a->n_heads * ((a->vdim + 31) / 32) > 148 ? 2 : 1;
+    // A warp is four row slices x eight lanes, a lane owns one or two columns: the choice of the linear-attention scan. Without the
+    // correction a CTA with one column per lane takes about 0.6 of the time of one with two; the busiest SM decides.
+    const int64_t c1 = (int64_t)a->n_seqs * a->n_heads * ((a->vdim + 31) / 32), c2 = (int64_t)a->n_seqs * a->n_heads * ((a->vdim + 63) / 64);
+    int rs = 4, nc = (DELTA ? c1 > 148 : 10 * ((c2 + 147) / 148) <= 6 * ((c1 + 147) / 148)) ? 2 : 1;
     if (a->rs_force == 2 || a->rs_force == 4) { rs = a->rs_force; nc = 1; }
     if (a->rs_force == 8) { rs = 4; nc = 2; }
     if (a->dim > 256) { rs = 4; nc = 1; }                    // 128 rows per thread, 16 tokens per round
