@@ -426,13 +426,24 @@ __global__ void __launch_bounds__(128, MINB) attn_window_prefill_mma_kernel(p3_a
         const float l = half ? l1 : l0;
         const float gate = (a.gate ? a.gate[(size_t)(row0 + row) * a.n_heads + h] : 1.f) * (a.out_scale != 0.f ? a.out_scale : 1.f);
         const float inv = sig ? gate : (l > 0.f ? gate / l : 0.f);
+        float2 eg[DN];                                       // element-wise gates: all loads before the first store
+        if (a.elem_gate) {
+            const float* gr = a.elem_gate + (size_t)(row0 + row) * a.ld_elem_gate + (size_t)h * a.vdim + vc0 + tig * 2;
+            const bool pairs = a.ld_elem_gate % 2 == 0 && ((uintptr_t)a.elem_gate & 7) == 0;
+#pragma unroll
+            for (int n = 0; n < DN; n++) {
+                if (n * 8 + tig * 2 >= dv) eg[n] = make_float2(0.f, 0.f);
+                else if (pairs) eg[n] = *reinterpret_cast<const float2*>(gr + n * 8);
+                else eg[n] = make_float2(gr[n * 8], gr[n * 8 + 1]);
+            }
+        }
 #pragma unroll
         for (int n = 0; n < DN; n++) {
             const int c = n * 8 + tig * 2;
             if (c < dv) {
-                const size_t oc = (size_t)h * a.vdim + vc0 + c;
-                *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + row) * a.ld_out + c) =
-                    pack_bf16(o[n][half * 2] * inv * elem_gate(a, row0 + row, oc), o[n][half * 2 + 1] * inv * elem_gate(a, row0 + row, oc + 1));
+                float g0 = inv, g1 = inv;
+                if (a.elem_gate) { g0 *= 1.0f / (1.0f + expf(-eg[n].x)); g1 *= 1.0f / (1.0f + expf(-eg[n].y)); }
+                *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + row) * a.ld_out + c) = pack_bf16(o[n][half * 2] * g0, o[n][half * 2 + 1] * g1);
             }
         }
     }
