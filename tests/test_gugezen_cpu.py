@@ -190,7 +190,7 @@ def test_oracle_state_space_mixer_against_a_token_loop():
     for t in range(T):
         z, dt = p[t, :inner], p[t, inner + C:]
         c = w['p.conv.b'].clone()
-        for j in range(taps):                                 # the last column of the taps is the current token's
+        for j in range(taps):                                 # taps[:, -1] meets token t itself
             if t - j >= 0:
                 c = c + w['p.conv'][:, taps - 1 - j] * p[t - j, inner:inner + C]
         c = c / (1 + torch.exp(-c))
@@ -201,7 +201,7 @@ def test_oracle_state_space_mixer_against_a_token_loop():
             step = torch.log(1 + torch.exp(dt[hh] + w['p.dt_bias'][hh]))
             S[hh] = torch.exp(-torch.exp(w['p.A_log'][hh]) * step) * S[hh] + step * B[:, None] * x[None, :]
             y[hh * dv:(hh + 1) * dv] = Cc @ S[hh] + w['p.D'][hh] * x
-        y = y * z / (1 + torch.exp(-z))                       # the gate comes before the norm
+        y = y * z / (1 + torch.exp(-z))                       # gated first, normed in parts after that
         n = inner // parts
         rows.append(torch.cat([y[i * n:(i + 1) * n] / torch.sqrt((y[i * n:(i + 1) * n] ** 2).mean() + eps) for i in range(parts)]) * w['p.norm'])
     assert torch.allclose(O.mamba2(h, w, 'p.', mc, eps), torch.stack(rows) @ w['p.o'].T)
